@@ -1,4 +1,7 @@
-"""ctypes binding of libllamatov_b200.so (the C ABI declared in include/llamatov_b200.h).
+"""ctypes binding of libllamatov_b200.so (the C ABI declared in include/llamatov_b200.h) and of
+libllamatov_b200_dense.so (include/llamatov_b200_dense.h).  Each is loaded when one of its entry
+points is first called; both share errors, status word and launch counter through
+libllamatov_b200_common.so.
 
 There is no CPU fallback: if the shared library is missing or a call fails, a RuntimeError
 is raised with the library's own error text.
@@ -8,7 +11,11 @@ import os
 
 _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_HERE, "libllamatov_b200.so")
+COMMON_PATH = os.path.join(_HERE, "libllamatov_b200_common.so")
+DENSE_PATH = os.path.join(_HERE, "libllamatov_b200_dense.so")
 _lib = None
+_common = None
+_dense = None
 
 LT_OK = 0
 STATUS_BITS = {1: "kv_overflow", 2: "bad_length", 4: "bad_token", 8: "wait_timeout"}
@@ -78,33 +85,108 @@ _QUERIES = {"lt_attn_decode_batch_scratch_floats": ([_i, _i, _i], ctypes.c_long)
             "lt_set_chained_launch": ([_i], ctypes.c_int)}
 
 
+# ---- include/llamatov_b200_dense.h
+DN_MAX_SEG = 6
+DN_STORE, DN_RESID, DN_GLU = 0, 1, 2
+DN_ACT = {None: 0, "silu": 1, "sigmoid": 2, "logsigmoid": 3}
+DN_IN_TYPED, DN_IN_CAST, DN_IN_NORM = 0, 1, 2
+
+
+class DnEpilogue(ctypes.Structure):
+    _fields_ = [("kind", _i), ("out_f32", _i), ("nseg", _i), ("seg_end", _i * DN_MAX_SEG), ("seg_act", _i * DN_MAX_SEG),
+                ("seg_scale", _f * DN_MAX_SEG), ("bias", _vp), ("ls", _vp)]
+
+
+class DnPrologue(ctypes.Structure):
+    _fields_ = [("kind", _i), ("n1", _i), ("group", _i), ("count", _i), ("eps", _f), ("x", _vp), ("x2", _vp), ("w", _vp),
+                ("w_period", _i), ("gate", _vp)]
+
+
+class DnDecay(ctypes.Structure):
+    _fields_ = [("decay", _vp), ("la", _vp), ("ldla", _i), ("a1", _vp), ("a2", _vp), ("lda2", _i), ("rank", _i),
+                ("bias", _vp), ("inv_tau", _f)]
+
+
+class DnLatent(ctypes.Structure):
+    _fields_ = [(n, _i) for n in ("H", "dp", "rtp", "dvp", "rot", "rp", "rank", "window", "cap")] + \
+               [("scale", _f), ("eps", _f), ("freq", _vp), ("cnorm", _vp)]
+
+
+DENSE_SIGNATURES = {
+    "lt_dn_embed": [_vp, _i, _i, _vp, _f, _vp, _vp, _i, _i, _i, _i, _vp],
+    "lt_dn_norm_rows": [_vp, _i, _vp, _vp, _i, _vp, _i, _vp, _i, _i, _i, _i, _i, _i, _f, _vp],
+    "lt_dn_concat_rows": [_vp, _i, _i, _vp, _i, _i, _vp, _i, _i, _i, _vp],
+    "lt_dn_linear": [_vp, _i, _vp, _i, _vp, _i, _i, _i, _i, _i, ctypes.POINTER(DnEpilogue), _i, _vp],
+    "lt_dn_gemv": [_vp, _i, _vp, _i, _i, _i, ctypes.POINTER(DnPrologue), ctypes.POINTER(DnEpilogue), _vp],
+    "lt_dn_recurrence": [_vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, ctypes.POINTER(DnDecay), _vp],
+    "lt_dn_latent_rows": [_vp, _i, _vp, _vp, _i, _i, _i, _i, ctypes.POINTER(DnLatent), _vp],
+    "lt_dn_window_attn": [_vp, _i, _vp, _i, _vp, _i, _vp, _i, _vp, _i, _i, _i, _i, ctypes.POINTER(DnLatent), _vp],
+    "lt_dn_latent_step": [_vp, _vp, _vp, _vp, _vp, _vp, _i, ctypes.POINTER(DnLatent), _i, _vp, _vp],
+}
+_DENSE_QUERIES = {"lt_dn_latent_step_ws": ([_i, _i, _i, _i], ctypes.c_long)}
+# what the common library exports (the Q8_0 library passes these through to its users as well)
+_COMMON_NAMES = ("lt_last_error", "lt_version", "lt_launch_count", "lt_set_chained_launch", "lt_device_status",
+                 "lt_graph_replay_token", "lt_token_record", "lt_quant_q8", "lt_silu_mul_quant", "lt_silu_mul", "lt_add",
+                 "lt_rmsnorm", "lt_rmsnorm_quant", "lt_rope", "lt_append_kv", "lt_incr_len", "lt_argmax_scratch_bytes",
+                 "lt_argmax", "lt_embed_q8")
+
+
+def _bind(L, names):
+    for name in names:
+        fn = getattr(L, name)
+        if name in SIGNATURES:
+            fn.argtypes, fn.restype = SIGNATURES[name], ctypes.c_int
+        elif name in _RESTYPES:
+            fn.argtypes, fn.restype = [], _RESTYPES[name]
+        else:
+            fn.argtypes, fn.restype = _QUERIES[name]
+
+
+def _load(path):
+    if not os.path.exists(path):
+        raise RuntimeError(
+            "%s is not built (%s). Run `python -m llamatov_b200.build`; "
+            "this package has no CPU or PyTorch fallback." % (os.path.basename(path), path))
+    return ctypes.CDLL(path)
+
+
 def lib():
-    """The loaded library (loads on first use)."""
+    """The loaded Q8_0 library (loads on first use)."""
     global _lib
     if _lib is None:
-        if not os.path.exists(LIB_PATH):
-            raise RuntimeError(
-                "libllamatov_b200.so is not built (%s). Run `python -m llamatov_b200.build`; "
-                "this package has no CPU or PyTorch fallback." % LIB_PATH)
-        L = ctypes.CDLL(LIB_PATH)
-        for name, args in SIGNATURES.items():
-            fn = getattr(L, name)
-            fn.argtypes = args
-            fn.restype = ctypes.c_int
-        for name, rt in _RESTYPES.items():
-            fn = getattr(L, name)
-            fn.argtypes = []
-            fn.restype = rt
-        for name, (args, rt) in _QUERIES.items():
-            fn = getattr(L, name)
-            fn.argtypes = args
-            fn.restype = rt
+        L = _load(LIB_PATH)
+        _bind(L, list(SIGNATURES) + list(_RESTYPES) + list(_QUERIES))
         _lib = L
     return _lib
 
 
+def common():
+    """The library that the other two share (loads on first use)."""
+    global _common
+    if _common is None:
+        L = _load(COMMON_PATH)
+        _bind(L, _COMMON_NAMES)
+        _common = L
+    return _common
+
+
+def dense():
+    """The library of the bf16 / fp32 models (loads on first use)."""
+    global _dense
+    if _dense is None:
+        L = _load(DENSE_PATH)
+        for name, args in DENSE_SIGNATURES.items():
+            fn = getattr(L, name)
+            fn.argtypes, fn.restype = args, ctypes.c_int
+        for name, (args, rt) in _DENSE_QUERIES.items():
+            fn = getattr(L, name)
+            fn.argtypes, fn.restype = args, rt
+        _dense = L
+    return _dense
+
+
 def last_error():
-    return lib().lt_last_error().decode("utf-8", "replace")
+    return common().lt_last_error().decode("utf-8", "replace")
 
 
 def check(rc, what=""):
@@ -114,15 +196,19 @@ def check(rc, what=""):
 
 
 def call(name, *args):
-    check(getattr(lib(), name)(*args), name)
+    if name in DENSE_SIGNATURES:
+        L = dense()
+    else:
+        L = common() if name in _COMMON_NAMES else lib()
+    check(getattr(L, name)(*args), name)
 
 
 def launch_count():
-    return int(lib().lt_launch_count())
+    return int(common().lt_launch_count())
 
 
 def device_status(stream=None):
     """Read and clear the device status word; returns the set of flag names."""
     v = ctypes.c_uint(0)
-    check(lib().lt_device_status(ctypes.byref(v), stream), "lt_device_status")
+    check(common().lt_device_status(ctypes.byref(v), stream), "lt_device_status")
     return {n for bit, n in STATUS_BITS.items() if v.value & bit}

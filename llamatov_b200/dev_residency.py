@@ -19,6 +19,7 @@ import numpy as np
 import torch
 
 from . import _lib
+from . import archs
 from . import fact_dispatch as fd
 from .fact_dispatch import Q8Weight
 
@@ -245,7 +246,31 @@ def _np(w):
 
 # --------------------------------------------------------------------------- KV cache
 
-class DeviceKVCache:
+class _PositionCounter:
+    """Length of a cache: the host mirror `length` and, where kernels read it, a device int."""
+    __slots__ = ()
+
+    def _ensure_len_ptr(self, seed=True):
+        """Device int holding the length.  seed=True writes the host mirror into it (never
+        during capture: the captured step advances it on the device)."""
+        if self.len_ptr is None:
+            self._len = torch.zeros(1, dtype=torch.int32, device="cuda")
+            self.len_ptr = ctypes.c_void_p(self._len.data_ptr())
+            seed = True
+        if seed:
+            if _capturing():
+                raise RuntimeError("length seeding during graph capture")
+            self._len.fill_(self.length)
+        return self.len_ptr
+
+    def reset(self):
+        """Empty the cache for the next sequence; its buffers (and so captured pointers) stay."""
+        self.length = 0
+        if self._len is not None:
+            self._len.zero_()
+
+
+class DeviceKVCache(_PositionCounter):
     """Per-layer fp32 K and V buffers [max_seq, nkv*hd], position-major, with a device-side
     length counter (bpd/lib/dev_residency.py:418-541)."""
     __slots__ = ("max_seq", "nkv", "hd", "width", "k_ptr", "v_ptr", "length", "elem_bytes", "len_ptr",
@@ -267,19 +292,6 @@ class DeviceKVCache:
 
     def _row_off(self, pos):
         return pos * self.width * self.elem_bytes
-
-    def _ensure_len_ptr(self, seed=True):
-        """Device int holding the length.  seed=True writes the host mirror into it (never
-        during capture: the captured step advances it on the device)."""
-        if self.len_ptr is None:
-            self._len = torch.zeros(1, dtype=torch.int32, device="cuda")
-            self.len_ptr = ctypes.c_void_p(self._len.data_ptr())
-            seed = True
-        if seed:
-            if _capturing():
-                raise RuntimeError("length seeding during graph capture")
-            self._len.fill_(self.length)
-        return self.len_ptr
 
     def incr_len_dev(self):
         _lib.call("lt_incr_len", self.len_ptr, _stream())
@@ -320,6 +332,42 @@ class DeviceKVCache:
 
     def free(self):
         self._k = None; self._v = None; self.k_ptr = None; self.v_ptr = None
+
+
+class DeviceLatentCache(_PositionCounter):
+    """Latent rows of windowed latent attention: a ring of `cap` rows of `width` elements, position p in row p % cap,
+    with a device-side length counter.  `cap` holds the window and the rows of one pass, so the sequence itself may
+    be of any length."""
+    __slots__ = ("cap", "width", "length", "len_ptr", "rows", "_len")
+
+    def __init__(self, cap, width, dtype):
+        self.cap, self.width = int(cap), int(width)
+        self.rows = torch.zeros((self.cap, self.width), dtype=dtype, device="cuda")
+        self.length = 0
+        self.len_ptr = None
+        self._len = None
+        self._ensure_len_ptr()
+
+    def free(self):
+        self.rows = None
+
+
+class DeviceRecurrentState(_PositionCounter):
+    """fp32 state of a linear-attention layer, [heads, value size, key size]; starts at zero."""
+    __slots__ = ("state", "length", "len_ptr", "_len")
+
+    def __init__(self, heads, vdim, dim):
+        self.state = torch.zeros((heads, vdim, dim), dtype=torch.float32, device="cuda")
+        self.length = 0
+        self.len_ptr = None
+        self._len = None
+
+    def reset(self):
+        super().reset()
+        self.state.zero_()
+
+    def free(self):
+        self.state = None
 
 
 # --------------------------------------------------------------------------- per-op launchers
@@ -533,7 +581,7 @@ def _ensure_argmax_buf():
     global _ARGMAX_BUF, _ARGMAX_PARTIALS
     if _ARGMAX_BUF is None:
         t = torch.zeros(1, dtype=torch.int32, device="cuda")
-        s = torch.empty(_lib.lib().lt_argmax_scratch_bytes(), dtype=torch.uint8, device="cuda")
+        s = torch.empty(_lib.common().lt_argmax_scratch_bytes(), dtype=torch.uint8, device="cuda")
         _ARGMAX_BUF = (ctypes.c_void_p(t.data_ptr()), t)
         _ARGMAX_PARTIALS = (ctypes.c_void_p(s.data_ptr()), s)
     return _ARGMAX_BUF[0]
@@ -586,6 +634,14 @@ def _ensure_logits_buf(E, w):
     return _LOGITS_BUF
 
 
+def _ensure_logits_n(n):
+    """Fixed logits buffer of n values."""
+    global _LOGITS_BUF
+    if _LOGITS_BUF is None or _LOGITS_BUF.n != n:
+        _LOGITS_BUF = DevTensor.empty((n,)); _LOGITS_BUF._owns = False
+    return _LOGITS_BUF
+
+
 def _ensure_logits_scratch(E):
     """(bpd/lib/dev_residency.py:1119-1127)"""
     global _LOGITS_RMS, _LOGITS_XQ, _LOGITS_XD
@@ -628,17 +684,15 @@ def forward_pass_resident(w, cfg, tok, positions, kv_cache):
     """One token through the device-resident layer loop; several tokens by recursion, one at
     a time, so prefill and decode share one arithmetic (bpd/lib/dev_residency.py:1328-1593).
     Returns logits [1, 1, V] (None while a graph is being captured)."""
-    nh, nkv = cfg["n_head"], cfg["n_head_kv"]
-    hd = cfg["n_embd"] // nh
-    nl = cfg["n_layers"]
+    A = archs.of(cfg)
     if tok.numel() > 1 and _BATCHED_PREFILL and not _capturing() and _DEVICE_EMBED is None:
         from . import prefill as _pf
         if _pf.supported(cfg, w):
             flat = tok.reshape(-1)
             last = None
-            for c0 in range(0, flat.numel(), _pf.MAX_ROWS):
-                last = _pf.prefill_resident(w, cfg, flat[c0:c0 + _pf.MAX_ROWS], kv_cache,
-                                            want_logits=c0 + _pf.MAX_ROWS >= flat.numel())
+            for c0 in range(0, flat.numel(), A.max_rows):
+                last = _pf.prefill_resident(w, cfg, flat[c0:c0 + A.max_rows], kv_cache,
+                                            want_logits=c0 + A.max_rows >= flat.numel())
             return last
     if tok.numel() > 1:
         toks = tok.reshape(-1).tolist(); poss = positions.reshape(-1).tolist()
@@ -646,49 +700,20 @@ def forward_pass_resident(w, cfg, tok, positions, kv_cache):
         for ti, pi in zip(toks, poss):
             last = forward_pass_resident(w, cfg, torch.tensor([ti]), torch.tensor([pi]), kv_cache)
         return last
-    E = cfg["n_embd"]
     capturing = _capturing()
-    _resid_in, _resid_carry = _ensure_resid(E)
-    if _DEVICE_EMBED is not None:
-        # on-device token loop: the row is gathered from the Q8_0 table by the token id that
-        # the previous step's argmax left in device memory
-        dWq, dWd, tok_ptr, V = _DEVICE_EMBED
-        _lib.call("lt_embed_q8", dWq, dWd, tok_ptr, _resid_in.ptr, E, V, _stream())
-    elif not capturing:
-        row = _embedding_row(w, int(tok.reshape(-1)[0]), E)
-        _memcpy_htod(_resid_in.ptr, row, E * 4)
-        torch.cuda.current_stream().synchronize()      # `row` is pageable host memory
-    x_resident = _resid_in
-    eps = cfg["norm_eps"]
-    theta = cfg["rope_theta"]
-    for il in range(nl):
-        p = f"blk.{il}"
-        xd = x_resident
-        hdv = rms_norm_dev(xd, _np(w[f"{p}.attn_norm.weight"]), eps)
-        qd, kd, vd = qkv_fused_dev(hdv, w, p)
-        cache = kv_cache[il]
+    x = A.embed_step(w, cfg, tok)
+    for run in A.runs(cfg):
+        cache = kv_cache[run.slot]
         if cache is None:
             if capturing:
                 raise RuntimeError("KV cache allocation during graph capture: seed() first")
-            cache = DeviceKVCache(_KV_MAX_SEQ, nkv, hd); kv_cache[il] = cache
-        lp = cache._ensure_len_ptr(seed=not capturing)
-        # position = length before the append; attention sees the length after it
-        rope_dev_qk_fused(qd.ptr, lp, nh, nkv, hd, theta)
-        cache.append_at_len_incr(kd.ptr, vd.ptr)
-        cache.length += 1
-        yd = attn_decode_from_cache_masked(qd.ptr, cache, nh, hd ** -0.5, lp, cache.max_seq)
-        xres = q8_linear_add_residual_dev(yd, w[f"{p}.attn_output.weight"], xd)
-        h2 = rms_norm_dev(xres, _np(w[f"{p}.ffn_norm.weight"]), eps)
-        g, u = gateup_fused_dev(h2, w, p)
-        q8_linear_add_residual_dev(g, w[f"{p}.ffn_down.weight"], xres, out=_resid_carry, silu_src=(g, u))
-        x_resident = _resid_carry
-        free_scratch()
-    _compute_folded_logits(w, cfg, E)
+            cache = A.new_cache(w, cfg, run); kv_cache[run.slot] = cache
+        x = A.layer_step(w, cfg, run, x, cache)
+    A.logits_step(w, cfg, x)
     if capturing:
         return None
     torch.cuda.synchronize()
-    lbuf = _ensure_logits_buf(E, w)
-    return torch.from_numpy(lbuf.to_host()).reshape(1, 1, lbuf.n)
+    return torch.from_numpy(_LOGITS_BUF.to_host()).reshape(1, 1, _LOGITS_BUF.n)
 
 
 def _compute_folded_logits(w, cfg, E):
@@ -925,6 +950,7 @@ class GraphRunner:
 
     def __init__(self, w, cfg, kv_cache):
         self.w = w; self.cfg = cfg; self.kv = kv_cache
+        self.arch = archs.of(cfg)
         self.E = cfg["n_embd"]
         self.graph = None
         self.captured = False
@@ -934,13 +960,11 @@ class GraphRunner:
     def seed(self, first_tok, first_pos):
         assert _GRAPH_PREP, "GraphRunner requires the device position/length path"
         assert_certified_composition()
-        _ensure_resid(self.E)
         if not _SLAB.enabled:
             raise RuntimeError("GraphRunner requires the slab arena (fixed pointers)")
         if _HOST_OPS:
             raise RuntimeError(f"GraphRunner cannot capture with host-op toggles active: {_HOST_OPS}")
-        _ensure_logits_buf(self.E, self.w)
-        _ensure_logits_scratch(self.E)
+        self.arch.ensure_buffers(self.w, self.cfg)
         _ensure_argmax_buf()
         if first_tok.numel() > 1:
             # the prompt but its last token in one batched pass; the last token takes the one-token
@@ -974,7 +998,8 @@ class GraphRunner:
         g = torch.cuda.CUDAGraph()
         torch.cuda.synchronize()
         n0 = _lib.launch_count()
-        self.fused = bool(_FUSED_STEP)
+        self.fused = bool(_FUSED_STEP) and self.arch.fused_step
+        self.argmax_in_step = self.fused
         self._tok_in = None
         if self.fused:
             # When the embedding table is a Q8_0 table (dequantising its blocks reproduces the rows the host
@@ -991,6 +1016,12 @@ class GraphRunner:
             n0 = _lib.launch_count()
             with torch.cuda.graph(g, stream=self.stream):
                 self._step_host.launch()
+        elif self.arch.device_token:
+            # the step gathers its embedding row by a token id in device memory and leaves the greedy token behind
+            self._tok_in = torch.zeros(1, dtype=torch.int32, device="cuda")
+            self.argmax_in_step = True
+            with torch.cuda.graph(g, stream=self.stream):
+                self._forward_on_device_token(self._tok_in, _ensure_argmax_buf())
         else:
             with torch.cuda.graph(g, stream=self.stream):
                 forward_pass_resident(self.w, self.cfg, tok, pos, self.kv)
@@ -1000,6 +1031,16 @@ class GraphRunner:
         self._assert_weight_cache_frozen()
         self.graph = g
         self.captured = True
+
+    def _forward_on_device_token(self, tok_dev, out_ptr):
+        """One step whose token id is read from `tok_dev`; its argmax goes to `out_ptr`."""
+        global _DEVICE_EMBED
+        _DEVICE_EMBED = (None, None, ctypes.c_void_p(tok_dev.data_ptr()), self.cfg.get("vocab"))
+        try:
+            forward_pass_resident(self.w, self.cfg, torch.tensor([0]), torch.tensor([0]), self.kv)
+            argmax_dev(_LOGITS_BUF.ptr, _LOGITS_BUF.n, out_ptr)
+        finally:
+            _DEVICE_EMBED = None
 
     def _q8_exact_table(self, probe_tok):
         """True if token_embd.weight is exactly representable as Q8_0 (checked on sample rows); uploads it."""
@@ -1057,6 +1098,8 @@ class GraphRunner:
         Call after seed().  `first_tok` is the token the first replay consumes."""
         global _DEVICE_EMBED
         self._assert_weight_cache_frozen()
+        if self.arch.device_token:
+            return self._capture_device_token_loop(first_tok, capacity)
         emb = _np(self.w["token_embd.weight"])
         _weights(emb)       # an untied table is not used by the host-driven step: upload it now
         self._weight_cache_frozen = (frozenset(_DEV_CONST.keys()), frozenset(fd._DEV_WEIGHT_CACHE.keys()),
@@ -1107,6 +1150,24 @@ class GraphRunner:
         self._assert_weight_cache_frozen()
         self.loop_graph = g
 
+    def _capture_device_token_loop(self, first_tok, capacity):
+        self._tok_dev = torch.tensor([int(first_tok)], dtype=torch.int32, device="cuda")
+        self._hist = torch.zeros(capacity, dtype=torch.int32, device="cuda")
+        self._step = torch.zeros(1, dtype=torch.int32, device="cuda")
+        self._hist_cap = capacity
+        lens = [c.length for c in self.kv]
+        g = torch.cuda.CUDAGraph()
+        torch.cuda.synchronize()
+        n0 = _lib.launch_count()
+        with torch.cuda.graph(g, stream=self.stream):
+            self._forward_on_device_token(self._tok_dev, self._tok_dev.data_ptr())
+            _lib.call("lt_token_record", self._tok_dev.data_ptr(), self._hist.data_ptr(), self._step.data_ptr(),
+                      capacity, _stream())
+        self.launches_per_step = _lib.launch_count() - n0
+        for c, n in zip(self.kv, lens):
+            c.length = n
+        self.loop_graph = g
+
     def reset_device_loop(self, first_tok):
         """Start the device loop over: next replay consumes `first_tok`, the token history is empty."""
         self.stream.synchronize()
@@ -1145,7 +1206,7 @@ class GraphRunner:
     def replay_token(self, tok):
         """Replay, device argmax, 4 bytes back to the host."""
         assert _LOGITS_BUF is not None, "replay_token requires device logits"
-        if self.fused and self._tok_in is not None and self.captured and self._raw_exec() is not None:
+        if self.argmax_in_step and self._tok_in is not None and self.captured and self._raw_exec() is not None:
             # token id up, graph, chosen token down, one wait: one call into the library
             self._ensure_pinned()
             self._pin_tok_np[0] = int(tok)
@@ -1157,7 +1218,7 @@ class GraphRunner:
             return int(self._pin_idx_np[0])
         self._launch(tok)
         ab = _ensure_argmax_buf()
-        if not self.fused:          # the fused step already left the argmax in the buffer
+        if not self.argmax_in_step:          # the fused step already left the argmax in the buffer
             with torch.cuda.stream(self.stream):
                 argmax_dev(_LOGITS_BUF.ptr, _LOGITS_BUF.n, ab)
         with torch.cuda.stream(self.stream):

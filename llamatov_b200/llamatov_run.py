@@ -4,6 +4,7 @@ GGUF parsing, tensor loading, `load_model`, `generate` and the command line -- w
 running on the device-resident engine of this package.
 
   python -m llamatov_b200.llamatov_run model.gguf 1,415,6557 20 --generate
+  python -m llamatov_b200.llamatov_run model_folder 1,415,6557 20 --dtype=bfloat16
 
 What is kept: `parse_gguf(path) -> (metadata, tensors, data_offset)` (bpd/llamatov_run.py:9-29),
 `lt(path, do, info)` (:497-511) for F32 / F16 / Q8_0 tensors, `dq8_0` (:184-207), the torch
@@ -15,8 +16,11 @@ since a block's largest element re-quantises to +-127 -- and `generate` decodes 
 `dev_residency.GraphRunner`; there is no CPU execution path here (device="cpu" is refused).
 Only the llama / qwen2 block structure with Q8_0 / F32 / F16 tensors is in scope; other tensor types
 and architectures of the reference's runner are refused with an error that says so.
+A folder with config.json and model.safetensors is read by the architecture its config names (`archs`).
 `write_gguf` is the inverse of the parser, for exporting synthetic models and for the tests.
 """
+import json
+import os
 import struct
 import sys
 import time
@@ -209,32 +213,47 @@ def _cfg_from(md):
                                md.get(f"{arch}.attention.layer_norm_epsilon", 1e-5))}
 
 
-def load_model(path, device="cuda", q8_blocks=True):
-    """(cfg, w) for `generate(..., preloaded=(cfg, w))` and the device-resident engine."""
+def load_folder(path, dtype="bfloat16"):
+    """(cfg, w) of a folder with config.json and model.safetensors; the architecture is the one the config names."""
+    from . import archs
+    from .safetensors_io import read_safetensors
+    with open(os.path.join(path, "config.json")) as f:
+        js = json.load(f)
+    A = archs.by_name(js.get("architecture"))
+    cfg = A.config_from_json(js, dtype)
+    return cfg, A.weights_from_safetensors(read_safetensors(os.path.join(path, "model.safetensors")), cfg)
+
+
+def load_model(path, device="cuda", q8_blocks=True, dtype="bfloat16"):
+    """(cfg, w) for `generate(..., preloaded=(cfg, w))` and the device-resident engine.  `dtype` is the element type of
+    models that are not quantised ("bfloat16" or "float32")."""
+    if os.path.isdir(path):
+        return load_folder(path, dtype)
     md, ts, do = parse_gguf(path)
     cfg = _cfg_from(md)
     w = {n: lt(path, do, info, q8_blocks=q8_blocks) for n, info in ts.items()}
     return cfg, w
 
 
-def generate(path, input_ids, n_tokens=20, device="cuda", preloaded=None, verbose=True):
+def generate(path, input_ids, n_tokens=20, device="cuda", preloaded=None, verbose=True, dtype="bfloat16"):
     """Greedy generation with the KV cache on the device: prompt prefill, one captured decode step,
     graph replays.  Returns the full id list (prompt + generated), like the reference."""
+    from . import archs
     from . import dev_residency as dr
     if device == "cpu":
         raise RuntimeError("llamatov_b200 has no CPU execution path; run the reference for device='cpu'")
     if not torch.cuda.is_available():
         raise RuntimeError("llamatov_b200.generate needs a CUDA device")
     t0 = time.time()
-    cfg, w = preloaded if preloaded is not None else load_model(path)
-    nl = cfg["n_layers"]
+    cfg, w = preloaded if preloaded is not None else load_model(path, dtype=dtype)
     if verbose:
         print(f"=== LlamaTov Generate ===\nModel: {path}")
-        print(f"Arch: {cfg['arch']}, layers: {nl}, heads: {cfg['n_head']}/{cfg['n_head_kv']}, embd: {cfg['n_embd']}")
+        heads = f", heads: {cfg['n_head']}/{cfg['n_head_kv']}" if "n_head" in cfg else ""
+        print(f"Arch: {cfg['arch']}, layers: {cfg['n_layers']}{heads}, embd: {cfg['n_embd']}")
         print(f"Loaded {len(w)} tensors in {time.time() - t0:.1f}s")
     dr.apply_production_profile()
     dr._KV_MAX_SEQ = max(dr._KV_MAX_SEQ, len(input_ids) + n_tokens + 1)
-    kv = [None] * nl
+    kv = [None] * archs.of(cfg).n_slots(cfg)
     runner = dr.GraphRunner(w, cfg, kv)
     generated = list(input_ids)
     t1 = time.time()
@@ -264,7 +283,8 @@ def main(argv=None):
     n = int(args[2]) if len(args) > 2 else 20
     if "--cpu" in argv:
         raise SystemExit("llamatov_b200 has no CPU execution path")
-    generate(p, ids, n)
+    dtype = next((a.split("=", 1)[1] for a in argv if a.startswith("--dtype=")), "bfloat16")
+    generate(p, ids, n, dtype=dtype)
 
 
 if __name__ == "__main__":
