@@ -119,11 +119,13 @@ DENSE_SIGNATURES = {
     "lt_dn_linear": [_vp, _i, _vp, _i, _vp, _i, _i, _i, _i, _i, ctypes.POINTER(DnEpilogue), _i, _vp],
     "lt_dn_gemv": [_vp, _i, _vp, _i, _i, _i, ctypes.POINTER(DnPrologue), ctypes.POINTER(DnEpilogue), _vp],
     "lt_dn_recurrence": [_vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, _i, ctypes.POINTER(DnDecay), _vp],
+    "lt_dn_recurrence_chunked": [_vp, _vp, _vp, _i, _vp, _vp, _i, _i, _i, _i, _i, ctypes.POINTER(DnDecay), _vp, _vp],
     "lt_dn_latent_rows": [_vp, _i, _vp, _vp, _i, _i, _i, _i, ctypes.POINTER(DnLatent), _vp],
     "lt_dn_window_attn": [_vp, _i, _vp, _i, _vp, _i, _vp, _i, _vp, _i, _i, _i, _i, ctypes.POINTER(DnLatent), _vp],
     "lt_dn_latent_step": [_vp, _vp, _vp, _vp, _vp, _vp, _i, ctypes.POINTER(DnLatent), _i, _vp, _vp],
 }
-_DENSE_QUERIES = {"lt_dn_latent_step_ws": ([_i, _i, _i, _i], ctypes.c_long)}
+_DENSE_QUERIES = {"lt_dn_latent_step_ws": ([_i, _i, _i, _i], ctypes.c_long),
+                  "lt_dn_recurrence_chunked_ws": ([_i, _i, _i, _i], ctypes.c_long)}
 # what the common library exports (the Q8_0 library passes these through to its users as well)
 _COMMON_NAMES = ("lt_last_error", "lt_version", "lt_launch_count", "lt_set_chained_launch", "lt_device_status",
                  "lt_graph_replay_token", "lt_token_record", "lt_quant_q8", "lt_silu_mul_quant", "lt_silu_mul", "lt_add",

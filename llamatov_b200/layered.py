@@ -15,12 +15,15 @@ Weights are packed once per model (`packed`): projections that read the same inp
 sizes and row lengths are padded to multiples of 8 with zeros, so kernels need no ragged edges.
 """
 import ctypes
-import math
 
 import torch
 
 from . import _lib, archs
 from . import dev_residency as dr
+
+# bf16 portions of at least this many tokens take the chunked form of the recurrence, for head sizes up to the limit
+CHUNKED_FROM = 64
+CHUNKED_MAX_DIM = 256
 
 DTYPES = {"bfloat16": torch.bfloat16, "float32": torch.float32}
 
@@ -167,11 +170,16 @@ class RecurrentMixer:
     def new_cache(self, cfg, max_rows):
         return dr.DeviceRecurrentState(self.H, self.dvp, self.dp)
 
-    def _recur(self, pk, y, ld, o, ldo, cache, T, dec):
+    def _recur(self, pk, y, ld, o, ldo, cache, T, dec, st=None):
         e = pk.esize
+        cache.length += T
+        if not pk.f32 and T >= CHUNKED_FROM and max(self.dp, self.dvp) <= CHUNKED_MAX_DIM:
+            ws = st.buf("chunk_ws", _lib.dense().lt_dn_recurrence_chunked_ws(T, self.H, self.dp, self.dvp), torch.float32)
+            _lib.call("lt_dn_recurrence_chunked", y, y + self.off_k * e, y + self.off_v * e, ld, cache.state.data_ptr(), o, ldo,
+                      T, self.H, self.dp, self.dvp, ctypes.byref(dec), ws, dr._stream())
+            return
         _lib.call("lt_dn_recurrence", y, y + self.off_k * e, y + self.off_v * e, ld, cache.state.data_ptr(), o, ldo, pk.f32,
                   T, self.H, self.dp, self.dvp, ctypes.byref(dec), dr._stream())
-        cache.length += T
 
     def step(self, pk, x, norm1, cache):
         b, e = pk.step, pk.esize
@@ -203,7 +211,7 @@ class RecurrentMixer:
                 dec.decay = self.decay.data_ptr()
             else:
                 dec.la, dec.ldla = la + b * T * self.nk * 4, self.nk
-            self._recur(pk, y + b * T * w * e, w, o + b * T * self.nv * 4, self.nv, c, T, dec)
+            self._recur(pk, y + b * T * w * e, w, o + b * T * self.nv * 4, self.nv, c, T, dec, st)
         self.norm.rows(o, self.nv, on, self.nv, pk.f32, R, self.nv, gate=y + self.off_g * e, ldg=w)
         self.out.rows(on, self.nv, st.x, st.ldx, R, self.epi_out)
 
