@@ -288,6 +288,16 @@ def run_config0(args):
     print(json.dumps(out))
 
 
+def run_layered(args):
+    """Mixer-layer models (bf16) beside the Q8_0 llama block at equal size: one JSON line."""
+    from llamatov_b200 import measure_layered
+    sampler = ClockSampler(0); sampler.start()
+    out = measure_layered.run(sizes=args.layered.split(","))
+    out["clocks"] = sampler.stop()
+    out["metric"] = "prefill and decode tok/s, one sequence, random weights"
+    print(json.dumps(out))
+
+
 def run_tp_leg(rank, world, steps):
     """BASELINE config 4 on the ranks of this run: Llama-3-8B-architecture random-init Q8_0 decode, TP = world,
     KV caches pre-filled to 4096 positions, batch 1 (attention in the declared split order, S = 16) and batch 32
@@ -320,6 +330,9 @@ def main():
     ap.add_argument("--no-tp", action="store_true", help="skip the tensor-parallel leg (the `tp` object)")
     ap.add_argument("--tp-steps", type=int, default=32)
     ap.add_argument("--config0", action="store_true", help="the single-GEMV case (BASELINE config 0) instead of decode")
+    ap.add_argument("--layered", nargs="?", const="0.5b,3b,8b", default=None, metavar="SIZES",
+                    help="prefill / decode throughput and kernel times of the mixer-layer models beside the Q8_0 llama "
+                         "block at equal size, instead of the headline workload")
     ap.add_argument("--step-mode", default=None, choices=["pdl", "persistent", "per-op"],
                     help="how the captured decode step is built (default: the engine's default)")
     args = ap.parse_args()
@@ -331,6 +344,10 @@ def main():
     if args.config0:
         if rank == 0:
             run_config0(args)
+        return
+    if args.layered:
+        if rank == 0:
+            run_layered(args)
         return
     if args.warmup < 3:
         args.warmup = 3

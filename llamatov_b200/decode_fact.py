@@ -13,6 +13,7 @@ import time
 
 import torch
 
+from . import archs
 from . import dev_residency as dr
 from . import fact_dispatch as fd
 from . import llamatov_run as R
@@ -34,6 +35,8 @@ def fp32lin(h, w, b=None):
 def load_model(path):
     """Parse GGUF, build cfg, load tensors; Q8_0 matrices stay Q8_0 blocks."""
     cfg, w = R.load_model(path)
+    if "n_head" not in cfg:        # not the llama / qwen2 block: the architecture's own configuration
+        return cfg, w
     cfg = {k: cfg[k] for k in ("n_layers", "n_head", "n_head_kv", "n_embd", "rope_theta", "norm_eps", "arch")}
     return cfg, w
 
@@ -59,11 +62,11 @@ def decode(path, input_ids, n_tokens=10, mode="int8", preloaded=None):
     if mode != "int8":
         raise NotImplementedError("decode: mode='int8' only")
     cfg, w = preloaded if preloaded is not None else load_model(path)
-    nl = cfg["n_layers"]
-    print(f"Arch {cfg['arch']} layers {nl} heads {cfg['n_head']}/{cfg['n_head_kv']} embd {cfg['n_embd']}", flush=True)
+    heads = f" heads {cfg['n_head']}/{cfg['n_head_kv']}" if "n_head" in cfg else ""
+    print(f"Arch {cfg['arch']} layers {cfg['n_layers']}{heads} embd {cfg['n_embd']}", flush=True)
     dr.apply_production_profile()
     dr._KV_MAX_SEQ = max(dr._KV_MAX_SEQ, len(input_ids) + n_tokens + 1)
-    kv_cache = [None] * nl
+    kv_cache = [None] * archs.of(cfg).n_slots(cfg)
     generated = list(input_ids)
     step_times = []
     for step in range(n_tokens):

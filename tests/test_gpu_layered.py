@@ -241,6 +241,14 @@ def test_generate_from_a_folder_is_greedy(tmp_path, plen):
     assert got[:plen] == prompt and len(got) == plen + 25
 
 
+def test_eager_driver_generates_the_same(tmp_path):
+    from llamatov_b200 import decode_fact
+    cfg = U.config()
+    path = U.write_model(tmp_path / "m", cfg, U.random_tensors(cfg, seed=26))
+    prompt = _tokens(cfg, 12, 3)
+    assert decode_fact.decode(path, prompt, 8) == R.generate(path, prompt, 8, verbose=False)
+
+
 def test_device_token_loop_equals_host_loop():
     cfg = U.config()
     c, w = U.product(cfg, U.random_tensors(cfg, seed=22), "bfloat16")
