@@ -13,7 +13,8 @@ namespace lt {
 namespace dn {
 
 constexpr int CH = 64;
-constexpr float SAFE_EXP = 60.0f;
+constexpr float LOG2E = 1.4426950408889634f;   // the kernels keep log decays to base 2
+constexpr float SAFE_EXP = 86.0f;              // of 2 (e^60)
 
 struct ChunkP {
     const bf16 *q, *k, *v;
@@ -65,6 +66,7 @@ __device__ __forceinline__ void load_logs(float* dst, int stride, const float* l
         const int t = e / nu, c = e - t * nu;
         float4 v = make_float4(0, 0, 0, 0);
         if (t0 + t < T) v = *(const float4*)(la + (long)(t0 + t) * ldla + c * 4);
+        v.x *= LOG2E; v.y *= LOG2E; v.z *= LOG2E; v.w *= LOG2E;
         *(float4*)(dst + t * stride + c * 4) = v;
     }
 }
@@ -93,13 +95,13 @@ __global__ void __launch_bounds__(256) k_chunk_state(const __grid_constant__ Chu
             float s = 0.0f;
             for (int j = CH - 1; j >= (seg + 1) * 16; j--) s += sla[j * P.dp + c];
             for (int j = seg * 16 + 15; j >= seg * 16; j--) {
-                const float x = to_f(sh[j * ks + c]) * expf(s);
+                const float x = to_f(sh[j * ks + c]) * exp2f(s);
                 const bf16 hi = from_f<bf16>(x);
                 sh[j * ks + c] = hi;
                 sl[j * ks + c] = from_f<bf16>(x - to_f(hi));
                 s += sla[j * P.dp + c];
             }
-            if (seg == 0) P.dend[((long)chunk * P.H + h) * P.dp + c] = expf(s);
+            if (seg == 0) P.dend[((long)chunk * P.H + h) * P.dp + c] = exp2f(s);
         }
     } else {
         const float lam = P.decay[h];
@@ -289,9 +291,9 @@ __global__ void __launch_bounds__(256, 2) k_chunk_out(const __grid_constant__ Ch
                     const float rb[4] = {bb.x, bb.y, bb.z, bb.w};
 #pragma unroll
                     for (int i = 0; i < 4; i++) {
-                        qa.x[i] *= expf(ra[i]);
-                        qb.x[i] *= expf(rb[i]);
-                        kq.x[i] *= expf(rk[i]);
+                        qa.x[i] *= exp2f(ra[i]);
+                        qb.x[i] *= exp2f(rb[i]);
+                        kq.x[i] *= exp2f(rk[i]);
                     }
                     unsigned ah[4], al[4], bh[2], bl2[2];
                     c_split2(qa.x[0], qa.x[1], ah[0], al[0]);
@@ -318,7 +320,7 @@ __global__ void __launch_bounds__(256, 2) k_chunk_out(const __grid_constant__ Ch
                 if (j > t) continue;
                 float s = 0.0f;
                 for (int c = 0; c < P.dp; c++)
-                    s = fmaf(to_f(sq[t * qs + c]) * to_f(sk[j * qs + c]), expf(sb[t * bs + c] - sb[j * bs + c]), s);
+                    s = fmaf(to_f(sq[t * qs + c]) * to_f(sk[j * qs + c]), exp2f(sb[t * bs + c] - sb[j * bs + c]), s);
                 acc[i] = s;
             }
         }
@@ -365,8 +367,8 @@ __global__ void __launch_bounds__(256, 2) k_chunk_out(const __grid_constant__ Ch
                     Quad qa = load_quad(sq + t * qs + c), qb = load_quad(sq + (t + 8) * qs + c);
                     const float4 ba = *(const float4*)(sb + t * bs + c), bb = *(const float4*)(sb + (t + 8) * bs + c);
                     const float4 p = *(const float4*)(sp + (mt + m) * bs + c);
-                    qa.x[0] *= expf(p.x + ba.x); qa.x[1] *= expf(p.y + ba.y); qa.x[2] *= expf(p.z + ba.z); qa.x[3] *= expf(p.w + ba.w);
-                    qb.x[0] *= expf(p.x + bb.x); qb.x[1] *= expf(p.y + bb.y); qb.x[2] *= expf(p.z + bb.z); qb.x[3] *= expf(p.w + bb.w);
+                    qa.x[0] *= exp2f(p.x + ba.x); qa.x[1] *= exp2f(p.y + ba.y); qa.x[2] *= exp2f(p.z + ba.z); qa.x[3] *= exp2f(p.w + ba.w);
+                    qb.x[0] *= exp2f(p.x + bb.x); qb.x[1] *= exp2f(p.y + bb.y); qb.x[2] *= exp2f(p.z + bb.z); qb.x[3] *= exp2f(p.w + bb.w);
                     c_split2(qa.x[0], qa.x[1], ah[0], al[0]);
                     c_split2(qb.x[0], qb.x[1], ah[1], al[1]);
                     c_split2(qa.x[2], qa.x[3], ah[2], al[2]);

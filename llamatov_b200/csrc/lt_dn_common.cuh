@@ -53,6 +53,12 @@ __device__ __forceinline__ float logsigmoid_f(float z) { return fminf(z, 0.0f) -
 __device__ __forceinline__ float gelu_tanh_f(float z) {
     return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
+// the same where the result is rounded to bf16: fast exponential and division (relative error below 2^-20)
+__device__ __forceinline__ float silu_bf16(float v) { return __fdividef(v, 1.0f + __expf(-v)); }
+__device__ __forceinline__ float sigmoid_bf16(float v) { return __fdividef(1.0f, 1.0f + __expf(-v)); }
+__device__ __forceinline__ float gelu_tanh_bf16(float z) {      // (1 + tanh u) / 2 = 1 / (1 + e^(-2u))
+    return __fdividef(z, 1.0f + __expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
+}
 __device__ __forceinline__ float act_f(int act, float v) {
     if (act == LT_DN_ACT_SILU) return v * sigmoid_f(v);
     if (act == LT_DN_ACT_SIGMOID) return sigmoid_f(v);
@@ -78,6 +84,24 @@ __device__ __forceinline__ RowEpi row_epi(const lt_dn_epilogue& e, int n) {
     r.bias = e.bias != nullptr ? e.bias[n] : 0.0f;
     r.ls = e.ls != nullptr ? e.ls[n] : 1.0f;
     return r;
+}
+// act(v + bias) * scale of N values of one row, the branch on the activation outside the loop
+template <bool BF16_OUT, int N>
+__device__ __forceinline__ void epi_values(const RowEpi& r, float (&v)[N]) {
+#pragma unroll
+    for (int i = 0; i < N; i++) v[i] += r.bias;
+    if (r.act == LT_DN_ACT_SILU) {
+#pragma unroll
+        for (int i = 0; i < N; i++) v[i] = BF16_OUT ? silu_bf16(v[i]) : v[i] * sigmoid_f(v[i]);
+    } else if (r.act == LT_DN_ACT_SIGMOID) {
+#pragma unroll
+        for (int i = 0; i < N; i++) v[i] = BF16_OUT ? sigmoid_bf16(v[i]) : sigmoid_f(v[i]);
+    } else if (r.act == LT_DN_ACT_LOGSIGMOID) {
+#pragma unroll
+        for (int i = 0; i < N; i++) v[i] = logsigmoid_f(v[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < N; i++) v[i] *= r.scale;
 }
 __device__ __forceinline__ float epi_value(const RowEpi& r, float v) { return act_f(r.act, v + r.bias) * r.scale; }
 

@@ -169,11 +169,24 @@ k_gemm_tc(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUten
                     for (int c = 0; c < 16; c += 4) reg_fence4(&v[a][c]);
                 if (row_ok) {
                     if (MA == 2) {
+                        float f[16];
+                        if (P.epi.out_f32) {
 #pragma unroll
-                        for (int c = 0; c < 16; c++)
-                            if (t0 + c0 + c < P.T)
-                                glu_store<bf16>(P.epi, P.Y, (long)(t0 + c0 + c) * P.ldy + row, __int_as_float(v[0][c]),
-                                                __int_as_float(v[MA - 1][c]));
+                            for (int c = 0; c < 16; c++)
+                                f[c] = gelu_tanh_f(__int_as_float(v[0][c])) * __int_as_float(v[MA - 1][c]);
+                            float* y = (float*)P.Y + (long)(t0 + c0) * P.ldy + row;
+#pragma unroll
+                            for (int c = 0; c < 16; c++)
+                                if (t0 + c0 + c < P.T) y[(long)c * P.ldy] = f[c];
+                        } else {
+#pragma unroll
+                            for (int c = 0; c < 16; c++)
+                                f[c] = gelu_tanh_bf16(__int_as_float(v[0][c])) * __int_as_float(v[MA - 1][c]);
+                            bf16* y = (bf16*)P.Y + (long)(t0 + c0) * P.ldy + row;
+#pragma unroll
+                            for (int c = 0; c < 16; c++)
+                                if (t0 + c0 + c < P.T) y[(long)c * P.ldy] = from_f<bf16>(f[c]);
+                        }
                     } else if (P.epi.kind == LT_DN_RESID) {
                         float* y = (float*)P.Y + (long)(t0 + c0) * P.ldy + row;
                         float old[16];
@@ -185,10 +198,22 @@ k_gemm_tc(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUten
                             if (t0 + c0 + c < P.T)
                                 y[(long)c * P.ldy] = fmaf(re.ls, __int_as_float(v[0][c]) + re.bias, old[c]);
                     } else {
+                        float f[16];
 #pragma unroll
-                        for (int c = 0; c < 16; c++)
-                            if (t0 + c0 + c < P.T)
-                                epi_store<bf16>(P.epi, re, P.Y, (long)(t0 + c0 + c) * P.ldy + row, __int_as_float(v[0][c]));
+                        for (int c = 0; c < 16; c++) f[c] = __int_as_float(v[0][c]);
+                        if (P.epi.out_f32) {
+                            epi_values<false>(re, f);
+                            float* y = (float*)P.Y + (long)(t0 + c0) * P.ldy + row;
+#pragma unroll
+                            for (int c = 0; c < 16; c++)
+                                if (t0 + c0 + c < P.T) y[(long)c * P.ldy] = f[c];
+                        } else {
+                            epi_values<true>(re, f);
+                            bf16* y = (bf16*)P.Y + (long)(t0 + c0) * P.ldy + row;
+#pragma unroll
+                            for (int c = 0; c < 16; c++)
+                                if (t0 + c0 + c < P.T) y[(long)c * P.ldy] = from_f<bf16>(f[c]);
+                        }
                     }
                 }
             }

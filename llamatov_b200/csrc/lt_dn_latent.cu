@@ -128,7 +128,7 @@ __global__ void __launch_bounds__(128) k_window_attn(const __grid_constant__ Win
     bf16* sK = sQ + WQ * ks;
     bf16* sV = sK + 2 * WK * ks;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    const int h = blockIdx.y, t0 = blockIdx.x * WQ, v0 = blockIdx.z * DV;
+    const int h = blockIdx.y, t0 = (gridDim.x - 1 - blockIdx.x) * WQ, v0 = blockIdx.z * DV;     // longest rows first
     const int c_n = P.dp >> 3, c_r = P.rtp >> 3, c_v = (min(DV, P.dvp - v0)) >> 3;
     const int qlast = min(t0 + WQ, P.T) - 1;
     const int jlo = max(0, P.np + t0 - P.window + 1), jhi = P.np + qlast;   // keys any query of the tile sees
@@ -352,6 +352,7 @@ template <typename T>
 __device__ __forceinline__ float row_dot8(const T* __restrict__ w, const float* x, int n, int g) {
     constexpr int N = Vec<T>::N;
     float a = 0.0f;
+#pragma unroll 4
     for (int c = g * N; c < n; c += 8 * N) {
         float f[N];
         Vec<T>::unpack(*(const uint4*)(w + c), f);
@@ -412,11 +413,29 @@ __global__ void __launch_bounds__(128) k_latent_prep(const __grid_constant__ Ste
         for (int j = L.rot + tid; j < L.rtp; j += 128) P.qr[h * L.rtp + j] = 0.0f;
     }
     __syncthreads();
-    const int g = tid & 7;
-    for (int r = blockIdx.y * 64 + (tid >> 3); r < min(L.rp, ((int)blockIdx.y + 1) * 64); r += 16) {
-        // rp is a multiple of 8 and 16 rows are in flight: whole warps may be past the end, half warps too
-        const float a = row_dot8<T>((const T*)P.ukT + ((long)h * L.rp + r) * L.dp, sm, L.dp, g);
-        if (g == 0) P.qa[h * L.rp + r] = a;
+    // eight lanes per row of W_uk^T, four rows per group of lanes, all in flight at once
+    const int g = tid & 7, r0 = blockIdx.y * 64 + (tid >> 3);
+    const T* w = (const T*)P.ukT + (long)h * L.rp * L.dp;
+    float a[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+    constexpr int N = Vec<T>::N;
+    for (int c = g * N; c < L.dp; c += 8 * N) {
+        uint4 v[4];
+#pragma unroll
+        for (int i = 0; i < 4; i++) v[i] = *(const uint4*)(w + (long)min(r0 + 16 * i, L.rp - 1) * L.dp + c);
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            float f[N];
+            Vec<T>::unpack(v[i], f);
+#pragma unroll
+            for (int j = 0; j < N; j++) a[i] = fmaf(f[j], sm[c + j], a[i]);
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        a[i] += __shfl_xor_sync(0xffffffffu, a[i], 1);
+        a[i] += __shfl_xor_sync(0xffffffffu, a[i], 2);
+        a[i] += __shfl_xor_sync(0xffffffffu, a[i], 4);
+        if (g == 0 && r0 + 16 * i < L.rp) P.qa[h * L.rp + r0 + 16 * i] = a[i];
     }
 }
 
@@ -441,11 +460,10 @@ __global__ void __launch_bounds__(128) k_latent_scan(const __grid_constant__ Ste
     const int per = (n + P.splits - 1) / P.splits;
     const int lo = pos - n + 1 + split * per, hi = min(pos + 1, lo + per);
 
-    for (int e = tid; e < SH * wr; e += 128) {
-        const int h = e / wr, c = e - h * wr;
-        float v = 0.0f;
-        if (h < nh) v = c < L.rp ? P.qa[(h0 + h) * L.rp + c] : P.qr[(h0 + h) * L.rtp + c - L.rp];
-        sQ[e] = v;
+    const int wq = wr >> 2;
+    for (int e = tid; e < SH * wq; e += 128) {
+        const int h = e / wq, c = (e - h * wq) * 4, hh = h0 + min(h, nh - 1);
+        cp16(sQ + h * wr + c, c < L.rp ? P.qa + hh * L.rp + c : P.qr + hh * L.rtp + c - L.rp, h < nh);
     }
     float acc[RD][SH][2];
 #pragma unroll
@@ -460,10 +478,9 @@ __global__ void __launch_bounds__(128) k_latent_scan(const __grid_constant__ Ste
         __syncthreads();
         for (int e = tid; e < SR * cu; e += 128) {
             const int r = e / cu, c = e - r * cu;
-            uint4 v = make_uint4(0, 0, 0, 0);
-            if (r < nr) v = ((const uint4*)((const T*)P.ring + (long)((p0 + r) % L.cap) * wr))[c];
-            *(uint4*)(sK + r * stride + c * N) = v;
+            cp16(sK + r * stride + c * N, (const T*)P.ring + (long)((p0 + min(r, nr - 1)) % L.cap) * wr + c * N, r < nr);
         }
+        asm volatile("cp.async.commit_group;\n\tcp.async.wait_group 0;" ::: "memory");
         __syncthreads();
         float s0 = 0.0f, s1 = 0.0f;
         const float* q0 = sQ + (2 * warp) * wr;
@@ -538,34 +555,57 @@ __global__ void __launch_bounds__(128) k_latent_scan(const __grid_constant__ Ste
     }
 }
 
-// CTA (h, y): combines the splits of head h, then 32 rows of the value projection
+// CTA (h, y): combines the splits of head h (two halves of the threads take two halves of the splits), then 32 rows of
+// the value projection
+constexpr int OT = 256;
 template <typename T>
-__global__ void __launch_bounds__(128) k_latent_out(const __grid_constant__ StepP P) {
+__global__ void __launch_bounds__(OT) k_latent_out(const __grid_constant__ StepP P) {
     extern __shared__ __align__(16) float sm[];
+    __shared__ float sred[OT / 32];
     const lt_dn_latent& L = P.L;
-    float* su = sm;            // [rp]
-    float* sw = sm + L.rp;     // [splits]
-    const int tid = threadIdx.x, h = blockIdx.x;
+    float* su = sm;                // [2][rp]
+    float* sw = sm + 2 * L.rp;     // [splits]
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.x;
     float m = -INFINITY;
-    for (int s = 0; s < P.splits; s++) m = fmaxf(m, P.pm[(long)s * L.H + h]);
-    float l = 0.0f;
-    for (int s = 0; s < P.splits; s++) l += P.pl[(long)s * L.H + h] * expf(P.pm[(long)s * L.H + h] - m);
-    const float inv = 1.0f / l;
-    for (int s = tid; s < P.splits; s += 128) sw[s] = expf(P.pm[(long)s * L.H + h] - m) * inv;
+    for (int s = tid; s < P.splits; s += OT) m = fmaxf(m, P.pm[(long)s * L.H + h]);
+    m = warp_max(m);
+    if (lane == 0) sred[warp] = m;
     __syncthreads();
-    for (int c = tid; c < L.rp; c += 128) {
-        float a = 0.0f;
-        for (int s = 0; s < P.splits; s++) a = fmaf(sw[s], P.pu[((long)s * L.H + h) * L.rp + c], a);
-        su[c] = a;
-    }
-    __syncthreads();
-    const int g = tid & 7;
 #pragma unroll
-    for (int k = 0; k < 2; k++) {
-        const int v = blockIdx.y * 32 + k * 16 + (tid >> 3);
-        const float a = row_dot8<T>((const T*)P.uv + ((long)h * L.dvp + min(v, L.dvp - 1)) * L.rp, su, L.rp, g);
-        if (g == 0 && v < L.dvp) ((T*)P.out)[h * L.dvp + v] = from_f<T>(a);
+    for (int i = 0; i < OT / 32; i++) m = fmaxf(m, sred[i]);
+    __syncthreads();
+    float l = 0.0f;
+    for (int s = tid; s < P.splits; s += OT) {
+        const float w = expf(P.pm[(long)s * L.H + h] - m);
+        sw[s] = w;
+        l = fmaf(w, P.pl[(long)s * L.H + h], l);
     }
+    l = warp_sum(l);
+    if (lane == 0) sred[warp] = l;
+    __syncthreads();
+    l = 0.0f;
+#pragma unroll
+    for (int i = 0; i < OT / 32; i++) l += sred[i];
+    const float inv = 1.0f / l;
+    const int half = tid >> 7, hs = (P.splits + 1) >> 1;
+    const int s0 = half * hs, s1 = min(P.splits, s0 + hs);
+    for (int c = (tid & 127) * 4; c < L.rp; c += 512) {
+        const float* u = P.pu + (long)h * L.rp + c;
+        float4 a = make_float4(0, 0, 0, 0);
+#pragma unroll 8
+        for (int s = s0; s < s1; s++) {
+            const float4 v = *(const float4*)(u + (long)s * L.H * L.rp);
+            const float w = sw[s];
+            a.x = fmaf(w, v.x, a.x); a.y = fmaf(w, v.y, a.y); a.z = fmaf(w, v.z, a.z); a.w = fmaf(w, v.w, a.w);
+        }
+        *(float4*)(su + half * L.rp + c) = make_float4(a.x * inv, a.y * inv, a.z * inv, a.w * inv);
+    }
+    __syncthreads();
+    for (int c = tid; c < L.rp; c += OT) su[c] += su[L.rp + c];
+    __syncthreads();
+    const int g = tid & 7, v = blockIdx.y * 32 + (tid >> 3);
+    const float a = row_dot8<T>((const T*)P.uv + ((long)h * L.dvp + min(v, L.dvp - 1)) * L.rp, su, L.rp, g);
+    if (g == 0 && v < L.dvp) ((T*)P.out)[h * L.dvp + v] = from_f<T>(a);
     if (h == 0 && blockIdx.y == 0 && tid == 0) *P.len += 1;     // nothing of this launch reads it
 }
 
@@ -591,7 +631,7 @@ static int launch_step(const StepP& P, cudaStream_t s) {
     else k_latent_scan<T, 4><<<grid, 128, smem, s>>>(P);
     rc = check_launch("lt_dn_latent_step (scan)");
     if (rc != LT_OK) return rc;
-    k_latent_out<T><<<dim3(L.H, (L.dvp + 31) / 32), 128, (L.rp + P.splits) * 4, s>>>(P);
+    k_latent_out<T><<<dim3(L.H, (L.dvp + 31) / 32), OT, (2 * L.rp + P.splits) * 4, s>>>(P);
     return check_launch("lt_dn_latent_step (out)");
 }
 
