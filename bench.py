@@ -33,6 +33,7 @@ With N > 1 every rank runs an independent replica of the model (the 0.5B model d
 shard: 2 KV heads, 0.5 GB of weights); value is the sum of tokens over ranks / max time.
 
 --impl reference times the CPU implementation on the host cores (rank 0 only).
+--layered times the mixer-layer models instead (llamatov_b200/measure_layered.py), beside the Q8_0 block at equal size.
 """
 import argparse
 import ctypes
