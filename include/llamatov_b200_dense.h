@@ -1,7 +1,7 @@
 /*
  * llamatov_b200_dense.h -- C ABI of libllamatov_b200_dense.so: the sm_100a kernels of models whose weights stay in
- * bfloat16 or fp32 and whose layers are mixers (linear-attention recurrences, windowed latent attention) with a
- * gated feed-forward.  Errors, the status word and the launch counter are those of libllamatov_b200_common.so
+ * bfloat16 or fp32 and whose layers are mixers (linear-attention and state-space recurrences, windowed latent attention,
+ * grouped-query attention) with a gated feed-forward.  Errors, the status word and the launch counter are those of libllamatov_b200_common.so
  * (llamatov_b200.h); the conventions of that header hold here too.
  *
  * Element type: `f32` = 0 means weights and activations are bfloat16 with fp32 accumulation, 1 means everything is
@@ -22,7 +22,12 @@ extern "C" {
 /* what a linear does with v = (W x)[n] (+ bias[n]) */
 #define LT_DN_STORE 0 /* y = act(v) * scale, per output segment */
 #define LT_DN_RESID 1 /* y (fp32) += ls[n] * v; ls may be NULL (1) */
-#define LT_DN_GLU 2   /* rows n and n + M of W are gate and up: y = gelu_tanh(v_gate) * v_up, M outputs */
+#define LT_DN_GLU 2   /* rows n and n + M of W are gate and up: y = glu(v_gate, v_up), M outputs */
+#define LT_DN_STORE_GLU 3 /* lt_dn_gemv only: rows below glu_from as LT_DN_STORE, then M - glu_from gate and as many up
+                             rows as LT_DN_GLU, whose outputs go to y2 */
+
+#define LT_DN_GLU_GELU 0    /* gelu_tanh(g) * u */
+#define LT_DN_GLU_CLAMPED 1 /* g = min(g, limit), u = clamp(u, -limit, limit): g * sigmoid(alpha g) * (u + 1) */
 
 #define LT_DN_ACT_NONE 0
 #define LT_DN_ACT_SILU 1
@@ -40,11 +45,18 @@ typedef struct {
     float seg_scale[LT_DN_MAX_SEG];
     const float* bias;            /* [M] or NULL */
     const float* ls;              /* [M] or NULL */
+    int glu_act;
+    float glu_alpha, glu_limit;
+    int tail_from, ldtail;        /* LT_DN_STORE with tail: outputs n >= tail_from go in fp32 to tail[t][n - tail_from] */
+    float* tail;                  /* or NULL */
+    int glu_from;
+    void* y2;
 } lt_dn_epilogue;
 
 #define LT_DN_IN_TYPED 0 /* x: K elements of the element type */
 #define LT_DN_IN_CAST 1  /* fp32 x [n1], then fp32 x2 [K - n1] (x2 may be NULL when n1 == K) */
-#define LT_DN_IN_NORM 2  /* fp32 x [K] in groups: x / sqrt(sum / count + eps) * w (* gate) */
+#define LT_DN_IN_NORM 2  /* fp32 x [n1] in groups: x / sqrt(sum / count + eps) * w (* gate), then K - n1 elements of the
+                            element type from x2 (n1 = 0 means K) */
 
 typedef struct {
     int kind;
@@ -52,20 +64,25 @@ typedef struct {
     int group, count;   /* LT_DN_IN_NORM: elements per group (padded) and how many of them count in the mean */
     float eps;
     const void* x;
-    const float* x2;
+    const void* x2;
     const float* w;     /* [w_period], index = position modulo w_period */
     int w_period;
-    const void* gate;   /* K elements of the element type, or NULL */
+    const void* gate;   /* n1 elements of the element type, or NULL */
+    int gate_first;     /* the gate multiplies x ahead of the norm instead of the normed value */
+    int seg, segp;      /* seg > 0: the vector is segments of segp elements of which seg are real, and a group is `count`
+                           consecutive real elements wherever the segments end (w has n1 entries then) */
 } lt_dn_prologue;
 
-/* x[t][0..ld) = table[tok[t]][0..E) * scale in fp32, zeros from E to ld; x0 (or NULL) gets the same rows. */
-int lt_dn_embed(const void* table, int f32, int tab_ld, const int* tok, float scale, float* x, float* x0, int E, int ld,
-                int V, int T, void* stream);
+/* x[t][0..ld) = table[tok[t]][0..E) * scale in fp32, zeros from E to ld; x0 (or NULL) gets the same rows.  With norm_w
+ * [E] (or NULL) the row is then RMS-normed: v / sqrt(mean(v^2) + eps) * norm_w. */
+int lt_dn_embed(const void* table, int f32, int tab_ld, const int* tok, float scale, const float* norm_w, float eps, float* x,
+                float* x0, int E, int ld, int V, int T, void* stream);
 
 /* rows of fp32 x in groups of `group` elements: y = x / sqrt(sum / count + eps) * w (* gate), stored in the element
- * type.  rows (or NULL): row t reads x row rows[t]. */
+ * type.  rows (or NULL): row t reads x row rows[t].  gate_first, seg, segp as in lt_dn_prologue. */
 int lt_dn_norm_rows(const float* x, int ldx, const int* rows, const float* w, int w_period, const void* gate, int ldg,
-                    void* y, int ldy, int f32, int T, int N, int group, int count, float eps, void* stream);
+                    void* y, int ldy, int f32, int T, int N, int group, int count, float eps, int gate_first, int seg, int segp,
+                    void* stream);
 
 /* y[t] = [x[t], x2[t]] cast to the element type, n1 and n2 columns */
 int lt_dn_concat_rows(const float* x, int ldx, int n1, const float* x2, int ldx2, int n2, void* y, int ldy, int f32, int T,
@@ -85,7 +102,8 @@ int lt_dn_gemv(const void* W, int ldw, void* Y, int f32, int M, int K, const lt_
  * q, k, v: element type, row stride ld, head h at columns h*dp (q, k) and h*dvp (v); o: fp32, row stride ldo.
  * The decay a_t comes from exactly one of: decay [H] (one constant per head); la [T][ldla] fp32, the logarithms per
  * key channel, head h at h*dp; or, for T = 1, a1 [rank] (element type) with a2 [H*dp][lda2], bias [H*dp]:
- * log a = logsigmoid(a2 a1 + bias) * inv_tau. */
+ * log a = logsigmoid(a2 a1 + bias) * inv_tau; or the state-space form, hla [T][ldh] fp32 with hdt [T][ldh] and D [H]:
+ *   S <- exp(hla_t) S + hdt_t k_t v_t^T,  o_t = S^T q_t + D v_t,   q and k shared by `per` consecutive heads. */
 typedef struct {
     const float* decay;
     const float* la;
@@ -95,12 +113,16 @@ typedef struct {
     int lda2, rank;
     const float* bias;
     float inv_tau;
+    const float* hla;
+    const float* hdt;
+    const float* D;
+    int ldh, per;
 } lt_dn_decay;
 
 int lt_dn_recurrence(const void* q, const void* k, const void* v, int ld, float* S, float* o, int ldo, int f32, int T,
                      int H, int dp, int dvp, const lt_dn_decay* h_decay, void* stream);
 
-/* The same over a prompt portion in chunks on the tensor cores (bf16 only; la or decay).  ws: fp32 workspace of
+/* The same over a prompt portion in chunks on the tensor cores (bf16 only; la, decay or hla).  ws: fp32 workspace of
  * lt_dn_recurrence_chunked_ws(T, H, dp, dvp) elements. */
 long lt_dn_recurrence_chunked_ws(int T, int H, int dp, int dvp);
 int lt_dn_recurrence_chunked(const void* q, const void* k, const void* v, int ld, float* S, float* o, int ldo, int T,
@@ -137,6 +159,62 @@ int lt_dn_window_attn(const void* q, int ldq, const void* kn, int ldkn, const vo
 long lt_dn_latent_step_ws(int H, int rp, int rtp, int splits);
 int lt_dn_latent_step(const void* y, void* ring, int* len, const void* ukT, const void* uv, void* out, int f32,
                       const lt_dn_latent* h_l, int splits, float* ws, void* stream);
+
+/* State-space mixer: a recurrence with step sizes per token and head, behind a short convolution.
+ * From `xbc` on a row holds C = H*dvp + 2*G*dp channels that pass a causal convolution of `taps` taps per channel and silu: x
+ * (H*dvp), then keys and queries of G groups (G*dp each).  The convolution's last inputs are kept in a ring [taps][C] of the
+ * element type, position p in row p % taps. */
+typedef struct {
+    int H, G, dp, dvp, taps;
+    const float* conv;     /* [taps][C]; the last tap is the current token's */
+    const float* conv_b;   /* [C] */
+    const float* dt_bias;  /* [H] */
+    const float* A;        /* [H]: log decay per unit of step size (negative) */
+    const float* D;        /* [H] */
+} lt_dn_ssd;
+
+/* T rows at positions pos0 ..: out [T][ldo] = silu(conv + bias), hdt = softplus(dt + dt_bias), hla = A * hdt ([T][H] fp32; dt
+ * [T][lddt] fp32); then the ring takes the portion's last inputs (two launches). */
+int lt_dn_ssd_rows(const void* xbc, int ld, const float* dt, int lddt, void* ring, void* out, int ldo, float* hla, float* hdt,
+                   int f32, int T, int pos0, const lt_dn_ssd* h_s, void* stream);
+
+/* One token at position *len (then *len += 1): convolution, step size and recurrence in one launch.  S [H][dvp][dp] fp32, o
+ * [H*dvp] fp32.  ticket: one int, zero between launches. */
+int lt_dn_ssd_step(const void* xbc, const float* dt, void* ring, float* S, float* o, int f32, int* len, int* ticket,
+                   const lt_dn_ssd* h_s, void* stream);
+
+/* Grouped-query attention over all earlier positions.  The cache keeps k [cap][G*dp] and v [cap][G*dvp] of the element
+ * type, position p in row p. */
+typedef struct {
+    int H, G, dp, dvp;     /* query heads, key/value heads, padded head sizes */
+    int rot;               /* rotated dimensions of a head: i is paired with i + rot/2 */
+    int qcount, kcount;    /* real elements of all queries / all keys (the norms' means) */
+    int cap;               /* rows of the cache */
+    float scale, softcap, eps;   /* softcap 0: none; else score <- softcap * tanh(score / softcap) */
+    float vmix;            /* v <- (1 - vmix) v + vmix * vfirst where vfirst is given */
+    const float* freq;     /* [rot/2][2]: a frequency as the sum of two floats */
+    const float* qnorm;    /* [H*dp] */
+    const float* knorm;    /* [G*dp] */
+} lt_dn_gqa;
+
+/* T rows at positions pos0 ..: y rows are [q: H*dp | k: G*dp | v: G*dvp ...], row stride ld.  Norms q and k over the whole
+ * projection, rotates them, mixes v; q is replaced, k and v go to the cache.  vfirst [T][G*dvp] or NULL: with vmix_store the
+ * row's own v is written there instead of being mixed. */
+int lt_dn_gqa_rows(void* y, int ld, void* kc, void* vc, void* vfirst, int vmix_store, int f32, int T, int pos0,
+                   const lt_dn_gqa* h_a, void* stream);
+
+/* out[t][h*dvp ..] = gate[t][h] * softmax over positions <= np + t of score(q, k) v for T queries at positions np .. (gate:
+ * fp32 or NULL). */
+int lt_dn_gqa_attn(const void* q, int ldq, const void* kc, const void* vc, const float* gate, int ldg, void* out, int ldo, int f32,
+                   int T, int np, const lt_dn_gqa* h_a, void* stream);
+
+/* One token at position *len (then *len += 1), in one launch: norms, rotation, value mixing, append, scores over `splits`
+ * ranges of positions per key head, combination, gate.  y: one row as in lt_dn_gqa_rows (not changed); gate [H] fp32 or NULL.
+ * ws: lt_dn_gqa_step_ws(H, dvp, splits) fp32 elements; tickets: lt_dn_gqa_step_tickets(H, G) ints, zero between launches. */
+long lt_dn_gqa_step_ws(int H, int dvp, int splits);
+int lt_dn_gqa_step_tickets(int H, int G);
+int lt_dn_gqa_step(const void* y, void* kc, void* vc, void* vfirst, int vmix_store, const float* gate, void* out, int f32, int* len,
+                   const lt_dn_gqa* h_a, int splits, float* ws, int* tickets, void* stream);
 
 #ifdef __cplusplus
 }

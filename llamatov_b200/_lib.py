@@ -87,24 +87,26 @@ _QUERIES = {"lt_attn_decode_batch_scratch_floats": ([_i, _i, _i], ctypes.c_long)
 
 # ---- include/llamatov_b200_dense.h
 DN_MAX_SEG = 6
-DN_STORE, DN_RESID, DN_GLU = 0, 1, 2
+DN_STORE, DN_RESID, DN_GLU, DN_STORE_GLU = 0, 1, 2, 3
+DN_GLU_GELU, DN_GLU_CLAMPED = 0, 1
 DN_ACT = {None: 0, "silu": 1, "sigmoid": 2, "logsigmoid": 3}
 DN_IN_TYPED, DN_IN_CAST, DN_IN_NORM = 0, 1, 2
 
 
 class DnEpilogue(ctypes.Structure):
     _fields_ = [("kind", _i), ("out_f32", _i), ("nseg", _i), ("seg_end", _i * DN_MAX_SEG), ("seg_act", _i * DN_MAX_SEG),
-                ("seg_scale", _f * DN_MAX_SEG), ("bias", _vp), ("ls", _vp)]
+                ("seg_scale", _f * DN_MAX_SEG), ("bias", _vp), ("ls", _vp), ("glu_act", _i), ("glu_alpha", _f), ("glu_limit", _f),
+                ("tail_from", _i), ("ldtail", _i), ("tail", _vp), ("glu_from", _i), ("y2", _vp)]
 
 
 class DnPrologue(ctypes.Structure):
     _fields_ = [("kind", _i), ("n1", _i), ("group", _i), ("count", _i), ("eps", _f), ("x", _vp), ("x2", _vp), ("w", _vp),
-                ("w_period", _i), ("gate", _vp)]
+                ("w_period", _i), ("gate", _vp), ("gate_first", _i), ("seg", _i), ("segp", _i)]
 
 
 class DnDecay(ctypes.Structure):
     _fields_ = [("decay", _vp), ("la", _vp), ("ldla", _i), ("a1", _vp), ("a2", _vp), ("lda2", _i), ("rank", _i),
-                ("bias", _vp), ("inv_tau", _f)]
+                ("bias", _vp), ("inv_tau", _f), ("hla", _vp), ("hdt", _vp), ("D", _vp), ("ldh", _i), ("per", _i)]
 
 
 class DnLatent(ctypes.Structure):
@@ -112,9 +114,18 @@ class DnLatent(ctypes.Structure):
                [("scale", _f), ("eps", _f), ("freq", _vp), ("cnorm", _vp)]
 
 
+class DnSsd(ctypes.Structure):
+    _fields_ = [(n, _i) for n in ("H", "G", "dp", "dvp", "taps")] + [(n, _vp) for n in ("conv", "conv_b", "dt_bias", "A", "D")]
+
+
+class DnGqa(ctypes.Structure):
+    _fields_ = [(n, _i) for n in ("H", "G", "dp", "dvp", "rot", "qcount", "kcount", "cap")] + \
+               [(n, _f) for n in ("scale", "softcap", "eps", "vmix")] + [(n, _vp) for n in ("freq", "qnorm", "knorm")]
+
+
 DENSE_SIGNATURES = {
-    "lt_dn_embed": [_vp, _i, _i, _vp, _f, _vp, _vp, _i, _i, _i, _i, _vp],
-    "lt_dn_norm_rows": [_vp, _i, _vp, _vp, _i, _vp, _i, _vp, _i, _i, _i, _i, _i, _i, _f, _vp],
+    "lt_dn_embed": [_vp, _i, _i, _vp, _f, _vp, _f, _vp, _vp, _i, _i, _i, _i, _vp],
+    "lt_dn_norm_rows": [_vp, _i, _vp, _vp, _i, _vp, _i, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _i, _i, _vp],
     "lt_dn_concat_rows": [_vp, _i, _i, _vp, _i, _i, _vp, _i, _i, _i, _vp],
     "lt_dn_linear": [_vp, _i, _vp, _i, _vp, _i, _i, _i, _i, _i, ctypes.POINTER(DnEpilogue), _i, _vp],
     "lt_dn_gemv": [_vp, _i, _vp, _i, _i, _i, ctypes.POINTER(DnPrologue), ctypes.POINTER(DnEpilogue), _vp],
@@ -123,8 +134,15 @@ DENSE_SIGNATURES = {
     "lt_dn_latent_rows": [_vp, _i, _vp, _vp, _i, _i, _i, _i, ctypes.POINTER(DnLatent), _vp],
     "lt_dn_window_attn": [_vp, _i, _vp, _i, _vp, _i, _vp, _i, _vp, _i, _i, _i, _i, ctypes.POINTER(DnLatent), _vp],
     "lt_dn_latent_step": [_vp, _vp, _vp, _vp, _vp, _vp, _i, ctypes.POINTER(DnLatent), _i, _vp, _vp],
+    "lt_dn_ssd_rows": [_vp, _i, _vp, _i, _vp, _vp, _i, _vp, _vp, _i, _i, _i, ctypes.POINTER(DnSsd), _vp],
+    "lt_dn_ssd_step": [_vp, _vp, _vp, _vp, _vp, _i, _vp, _vp, ctypes.POINTER(DnSsd), _vp],
+    "lt_dn_gqa_rows": [_vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, ctypes.POINTER(DnGqa), _vp],
+    "lt_dn_gqa_attn": [_vp, _i, _vp, _vp, _vp, _i, _vp, _i, _i, _i, _i, ctypes.POINTER(DnGqa), _vp],
+    "lt_dn_gqa_step": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _i, _vp, ctypes.POINTER(DnGqa), _i, _vp, _vp, _vp],
 }
-_DENSE_QUERIES = {"lt_dn_latent_step_ws": ([_i, _i, _i, _i], ctypes.c_long),
+_DENSE_QUERIES = {"lt_dn_gqa_step_ws": ([_i, _i, _i], ctypes.c_long),
+                  "lt_dn_gqa_step_tickets": ([_i, _i], _i),
+                  "lt_dn_latent_step_ws": ([_i, _i, _i, _i], ctypes.c_long),
                   "lt_dn_recurrence_chunked_ws": ([_i, _i, _i, _i], ctypes.c_long)}
 # what the common library exports (the Q8_0 library passes these through to its users as well)
 _COMMON_NAMES = ("lt_last_error", "lt_version", "lt_launch_count", "lt_set_chained_launch", "lt_device_status",

@@ -17,6 +17,7 @@ _REGISTRY = {
     "llama": "llamatov_b200.q8_block:ARCH",
     "qwen2": "llamatov_b200.q8_block:ARCH",
     "Nugusun": "llamatov_b200.layered:ARCH",
+    "Pakalix": "llamatov_b200.layered:PAKALIX",
 }
 
 

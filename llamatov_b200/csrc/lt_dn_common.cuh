@@ -49,6 +49,7 @@ struct Vec<float> {
 };
 
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float logsigmoid_f(float z) { return fminf(z, 0.0f) - log1pf(expf(-fabsf(z))); }
 __device__ __forceinline__ float gelu_tanh_f(float z) {
     return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
@@ -105,20 +106,45 @@ __device__ __forceinline__ void epi_values(const RowEpi& r, float (&v)[N]) {
 }
 __device__ __forceinline__ float epi_value(const RowEpi& r, float v) { return act_f(r.act, v + r.bias) * r.scale; }
 
+// output n of row t; Y has row stride ldy
 template <typename T>
-__device__ __forceinline__ void epi_store(const lt_dn_epilogue& e, const RowEpi& r, void* Y, long idx, float v) {
+__device__ __forceinline__ void epi_store(const lt_dn_epilogue& e, const RowEpi& r, void* Y, long t, int ldy, int n, float v) {
+    const long idx = t * ldy + n;
     if (e.kind == LT_DN_RESID) {
         float* y = (float*)Y + idx;
         *y = fmaf(r.ls, v + r.bias, *y);
+    } else if (e.tail != nullptr && n >= e.tail_from) {
+        e.tail[t * e.ldtail + n - e.tail_from] = epi_value(r, v);
     } else if (e.out_f32) {
         ((float*)Y)[idx] = epi_value(r, v);
     } else {
         ((T*)Y)[idx] = from_f<T>(epi_value(r, v));
     }
 }
+__device__ __forceinline__ float glu_f(const lt_dn_epilogue& e, float g, float u) {
+    if (e.glu_act == LT_DN_GLU_GELU) return gelu_tanh_f(g) * u;
+    g = fminf(g, e.glu_limit);
+    u = fminf(fmaxf(u, -e.glu_limit), e.glu_limit);
+    return g * sigmoid_f(e.glu_alpha * g) * (u + 1.0f);
+}
+// the same where the result is rounded to bf16, N values (bits of floats) with the branch outside the loop
+template <int N>
+__device__ __forceinline__ void glu_bf16(const lt_dn_epilogue& e, const int (&g)[N], const int (&u)[N], float (&f)[N]) {
+    if (e.glu_act == LT_DN_GLU_GELU) {
+#pragma unroll
+        for (int i = 0; i < N; i++) f[i] = gelu_tanh_bf16(__int_as_float(g[i])) * __int_as_float(u[i]);
+    } else {
+        const float lim = e.glu_limit, alpha = e.glu_alpha;
+#pragma unroll
+        for (int i = 0; i < N; i++) {
+            const float a = fminf(__int_as_float(g[i]), lim);
+            f[i] = __fdividef(a, 1.0f + __expf(-alpha * a)) * (fminf(fmaxf(__int_as_float(u[i]), -lim), lim) + 1.0f);
+        }
+    }
+}
 template <typename T>
 __device__ __forceinline__ void glu_store(const lt_dn_epilogue& e, void* Y, long idx, float g, float u) {
-    const float v = gelu_tanh_f(g) * u;
+    const float v = glu_f(e, g, u);
     if (e.out_f32) ((float*)Y)[idx] = v;
     else ((T*)Y)[idx] = from_f<T>(v);
 }
@@ -150,7 +176,9 @@ inline int sm_count() {
 // host checks shared by the launchers
 inline const char* epi_error(const lt_dn_epilogue* e) {
     if (e == nullptr) return "null epilogue";
-    if (e->kind < 0 || e->kind > LT_DN_GLU) return "unknown epilogue kind";
+    if (e->kind < 0 || e->kind > LT_DN_STORE_GLU) return "unknown epilogue kind";
+    if (e->glu_act < 0 || e->glu_act > LT_DN_GLU_CLAMPED) return "unknown gated activation";
+    if (e->tail != nullptr && (e->tail_from < 0 || e->ldtail < 1)) return "bad fp32 tail";
     if (e->nseg < 0 || e->nseg > LT_DN_MAX_SEG) return "too many segments";
     return nullptr;
 }

@@ -2,7 +2,7 @@
 //
 // bf16 (k_gemm_tc): tcgen05.mma kind::f16, fp32 accumulators in tensor memory.  A tile is MA x 128 weight rows (the
 // MMA's M: tensor-memory lanes) by NT tokens (its N: columns); with MA = 2 the second 128 rows are the "up" rows that
-// belong to the first 128 "gate" rows, so that gelu(gate) * up is formed where both accumulators are.  An epilogue
+// belong to the first 128 "gate" rows, so that act(gate) * up is formed where both accumulators are.  An epilogue
 // thread owns one weight row: bias, activation and layer scale are per-thread constants, and the 32 lanes of a
 // warp store 32 consecutive outputs of a token.
 //   warp 8 : producer, TMA tiles of 64 k (128-byte rows, hardware swizzle) into a ring of shared-memory stages
@@ -173,15 +173,13 @@ k_gemm_tc(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUten
                         if (P.epi.out_f32) {
 #pragma unroll
                             for (int c = 0; c < 16; c++)
-                                f[c] = gelu_tanh_f(__int_as_float(v[0][c])) * __int_as_float(v[MA - 1][c]);
+                                f[c] = glu_f(P.epi, __int_as_float(v[0][c]), __int_as_float(v[MA - 1][c]));
                             float* y = (float*)P.Y + (long)(t0 + c0) * P.ldy + row;
 #pragma unroll
                             for (int c = 0; c < 16; c++)
                                 if (t0 + c0 + c < P.T) y[(long)c * P.ldy] = f[c];
                         } else {
-#pragma unroll
-                            for (int c = 0; c < 16; c++)
-                                f[c] = gelu_tanh_bf16(__int_as_float(v[0][c])) * __int_as_float(v[MA - 1][c]);
+                            glu_bf16(P.epi, v[0], v[MA - 1], f);
                             bf16* y = (bf16*)P.Y + (long)(t0 + c0) * P.ldy + row;
 #pragma unroll
                             for (int c = 0; c < 16; c++)
@@ -201,7 +199,13 @@ k_gemm_tc(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUten
                         float f[16];
 #pragma unroll
                         for (int c = 0; c < 16; c++) f[c] = __int_as_float(v[0][c]);
-                        if (P.epi.out_f32) {
+                        if (P.epi.tail != nullptr && row >= P.epi.tail_from) {
+                            epi_values<false>(re, f);
+                            float* y = P.epi.tail + (long)(t0 + c0) * P.epi.ldtail + row - P.epi.tail_from;
+#pragma unroll
+                            for (int c = 0; c < 16; c++)
+                                if (t0 + c0 + c < P.T) y[(long)c * P.epi.ldtail] = f[c];
+                        } else if (P.epi.out_f32) {
                             epi_values<false>(re, f);
                             float* y = (float*)P.Y + (long)(t0 + c0) * P.ldy + row;
 #pragma unroll
@@ -335,7 +339,7 @@ __global__ void __launch_bounds__(256) k_gemm_f32(const float* __restrict__ W, i
             const int t = t0 + ty + 16 * j;
             if (t >= P.T) continue;
             if (GLU) glu_store<float>(P.epi, P.Y, (long)t * P.ldy + n, acc[0][i][j], acc[GLU ? 1 : 0][i][j]);
-            else epi_store<float>(P.epi, re, P.Y, (long)t * P.ldy + n, acc[0][i][j]);
+            else epi_store<float>(P.epi, re, P.Y, t, P.ldy, n, acc[0][i][j]);
         }
     }
 }
@@ -371,7 +375,9 @@ extern "C" int lt_dn_linear(const void* W, int ldw, const void* X, int ldx, void
     LT_REQUIRE(M > 0 && T > 0 && K > 0 && K % 8 == 0, "lt_dn_linear: M=%d T=%d K=%d (K a multiple of 8)", M, T, K);
     LT_REQUIRE(ldw >= K && ldw % 8 == 0 && ldx >= K && ldx % 8 == 0, "lt_dn_linear: ldw=%d ldx=%d must be multiples of 8, >= K=%d",
                ldw, ldx, K);
-    LT_REQUIRE(ldy >= M, "lt_dn_linear: ldy=%d < M=%d", ldy, M);
+    const int my = h_epi->kind == LT_DN_STORE && h_epi->tail != nullptr && h_epi->tail_from < M ? h_epi->tail_from : M;
+    LT_REQUIRE(ldy >= my, "lt_dn_linear: ldy=%d < M=%d", ldy, my);
+    LT_REQUIRE(h_epi->kind != LT_DN_STORE_GLU, "lt_dn_linear: the combined epilogue is lt_dn_gemv's");
     LT_REQUIRE(aligned16(W) && aligned16(X), "lt_dn_linear: W and X must be 16-byte aligned");
     LT_REQUIRE(variant == 0 || variant == 32 || variant == 64 || variant == 128 || variant == 256,
                "lt_dn_linear: unknown variant %d", variant);

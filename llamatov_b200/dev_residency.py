@@ -370,6 +370,48 @@ class DeviceRecurrentState(_PositionCounter):
         self.state = None
 
 
+class DeviceSsdState(DeviceRecurrentState):
+    """State of a state-space mixer: fp32 [heads, value size, key size], and a ring with the last `taps` inputs of its
+    convolution (position p in row p % taps; rows of positions that do not exist are never read)."""
+    __slots__ = ("ring",)
+
+    def __init__(self, heads, vdim, dim, taps, channels, dtype):
+        super().__init__(heads, vdim, dim)
+        self.ring = torch.zeros((taps, channels), dtype=dtype, device="cuda")
+        self._ensure_len_ptr()
+
+    def reset(self):
+        super().reset()
+        self.ring.zero_()
+
+    def free(self):
+        super().free()
+        self.ring = None
+
+
+class DeviceGroupedKV(_PositionCounter):
+    """Key and value rows of grouped-query attention in the model's element type, position p in row p of `cap`, with a
+    device-side length counter."""
+    __slots__ = ("cap", "k", "v", "length", "len_ptr", "_len")
+
+    def __init__(self, cap, kwidth, vwidth, dtype):
+        self.cap = int(cap)
+        self.k = torch.zeros((self.cap, kwidth), dtype=dtype, device="cuda")
+        self.v = torch.zeros((self.cap, vwidth), dtype=dtype, device="cuda")
+        self.length = 0
+        self.len_ptr = None
+        self._len = None
+        self._ensure_len_ptr()
+
+    def require(self, n):
+        """Raise unless n more positions fit."""
+        if self.length + n > self.cap:
+            raise RuntimeError(f"KV cache overflow: {self.length}+{n} > {self.cap}")
+
+    def free(self):
+        self.k = self.v = None
+
+
 # --------------------------------------------------------------------------- per-op launchers
 
 def _launch_quant(dX_ptr, dXq, dXd, K):

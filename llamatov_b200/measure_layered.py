@@ -10,7 +10,7 @@ import ctypes
 import numpy as np
 import torch
 
-from . import _lib, archs, layered
+from . import _lib, archs, dense_ops, layered
 from . import dev_residency as dr
 from . import prefill as pf
 from .fact_dispatch import Q8Weight
@@ -181,7 +181,7 @@ def kernel_times(s, T, only=None):
         Ws = [bf(rows, K) for _ in range(n)]
         Xs = [bf(T, K) for _ in range(n)]
         Y = torch.zeros(T, M, dtype=torch.float32 if kind == 1 else torch.bfloat16, **dev)
-        e = layered.epilogue(kind, segs=[(M, "silu", 1.0)] if kind == 0 else ())
+        e = dense_ops.epilogue(kind, segs=[(M, "silu", 1.0)] if kind == 0 else ())
         us = _chain_us([lambda W=W_, X=X_: _lib.call("lt_dn_linear", W.data_ptr(), K, X.data_ptr(), K, Y.data_ptr(), M, 0, M, K, T,
                                                      ctypes.byref(e), 0, st()) for W_, X_ in zip(Ws, Xs)])
         add(f"linear {name} {rows}x{K}, {T} rows", us, rows * K * 2 + T * K * 2 + T * M * (8 if kind == 1 else 2), 2.0 * rows * K * T, "q8 gemm")
@@ -203,11 +203,11 @@ def kernel_times(s, T, only=None):
         n = _copies(rows * K * 2)
         Ws = [bf(rows, K) for _ in range(n)]
         x, w = torch.randn(K, **dev), torch.ones(K)
-        nm = layered.Norm(w, K, K, 1e-6)
+        nm = dense_ops.Norm(w, K, K, 1e-6)
         xt = bf(K)
-        pro = layered.typed_input(xt.data_ptr()) if name == "down" else nm.prologue(x.data_ptr())
+        pro = dense_ops.typed_input(xt.data_ptr()) if name == "down" else nm.prologue(x.data_ptr())
         Y = torch.zeros(M, **dev)
-        e = layered.epilogue(kind, out_f32=True)
+        e = dense_ops.epilogue(kind, out_f32=True)
         us = _chain_us([lambda W=W_: _lib.call("lt_dn_gemv", W.data_ptr(), K, Y.data_ptr(), 0, M, K, ctypes.byref(pro), ctypes.byref(e), st())
                         for W_ in Ws])
         add(f"gemv {name} {rows}x{K}", us, rows * K * 2, 0, "q8 gemv")
@@ -300,7 +300,7 @@ def kernel_times(s, T, only=None):
     # ---- row operators
     if want("norm"):
         n = _copies(T * E * 4)
-        xs, w = [torch.randn(T, E, **dev) for _ in range(n)], layered.Norm(torch.ones(E), E, E, 1e-6)
+        xs, w = [torch.randn(T, E, **dev) for _ in range(n)], dense_ops.Norm(torch.ones(E), E, E, 1e-6)
         h = torch.empty(T, E, dtype=torch.bfloat16, **dev)
         us = _chain_us([lambda x=x_: w.rows(x.data_ptr(), E, h.data_ptr(), E, 0, T, E) for x_ in xs])
         add(f"norm rows {T}x{E}", us, T * E * 6, 0, "q8 rmsnorm")

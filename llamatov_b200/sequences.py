@@ -52,6 +52,9 @@ class Sequences:
         if V is not None and any(not 0 <= int(t) < V for t in tokens):
             raise ValueError("token id outside the vocabulary")
         s = self._slot(sid)
+        for c in s.kv:
+            if isinstance(c, dr.DeviceGroupedKV):
+                c.require(n)
         out = {}
         if n == 1:
             lg = self._one(s, int(tokens[0]))

@@ -9,7 +9,7 @@ import numpy as np
 import pytest
 import torch
 
-from llamatov_b200 import _lib, archs, dev_residency as dr, layered, llamatov_run as R, prefill as pf
+from llamatov_b200 import _lib, archs, dev_residency as dr, layered, llamatov_run as R, mixers, prefill as pf
 from llamatov_b200.sequences import Sequences
 from oracle import layered as L
 from tests import layered_util as U
@@ -102,7 +102,7 @@ def test_chunked_and_scanned_prompts_agree(monkeypatch):
     toks = _tokens(cfg, 200)
     S = Sequences(w, c)
     a = S.step("a", toks, range(200)).numpy()
-    monkeypatch.setattr(layered, "CHUNKED_FROM", 10 ** 9)
+    monkeypatch.setattr(mixers, "CHUNKED_FROM", 10 ** 9)
     b = S.step("b", toks, range(200)).numpy()
     assert U.rel_rms(a, b) < TOL["bfloat16"]
 

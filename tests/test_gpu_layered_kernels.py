@@ -5,7 +5,7 @@ import numpy as np
 import pytest
 import torch
 
-from llamatov_b200 import _lib, layered as P
+from llamatov_b200 import _lib, dense_ops as P
 from oracle import layered as L
 from tests.gpu_util import stream
 
@@ -147,10 +147,10 @@ def test_row_operators(f32):
     tab = _t((9, 13), 4, f32)
     tok = torch.tensor([8, 0, 3], dtype=torch.int32).cuda()
     a, b = torch.full((3, 16), 5.0).cuda(), torch.full((3, 16), 5.0).cuda()
-    _lib.call("lt_dn_embed", tab.data_ptr(), f32, 13, tok.data_ptr(), 3.5, a.data_ptr(), b.data_ptr(), 13, 16, 9, 3, stream())
+    _lib.call("lt_dn_embed", tab.data_ptr(), f32, 13, tok.data_ptr(), 3.5, None, 0.0, a.data_ptr(), b.data_ptr(), 13, 16, 9, 3, stream())
     _close(_np(a)[:, :13], _np(tab)[[8, 0, 3]] * 3.5, 1e-6)
     assert torch.equal(a, b) and (a[:, 13:] == 0).all()
-    _lib.call("lt_dn_embed", tab.data_ptr(), f32, 13, torch.tensor([9], dtype=torch.int32).cuda().data_ptr(), 1.0, a.data_ptr(), None, 13, 16,
+    _lib.call("lt_dn_embed", tab.data_ptr(), f32, 13, torch.tensor([9], dtype=torch.int32).cuda().data_ptr(), 1.0, None, 0.0, a.data_ptr(), None, 13, 16,
               9, 1, stream())
     assert _lib.device_status() == {"bad_token"}
     y = torch.empty(3, 40, dtype=DT[f32], device="cuda")

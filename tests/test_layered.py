@@ -100,7 +100,7 @@ def test_layer_runs(loop, want):
 
 
 def test_packing_pads_heads_and_columns():
-    from llamatov_b200 import layered as P
+    from llamatov_b200 import dense_ops as P
     W = torch.arange(2 * 5 * 3, dtype=torch.float32).reshape(10, 3)
     R = P._head_rows(W, [(2, 8), (3, 8)], 2)
     assert R.shape == (32, 3)
