@@ -33,7 +33,8 @@ With N > 1 every rank runs an independent replica of the model (the 0.5B model d
 shard: 2 KV heads, 0.5 GB of weights); value is the sum of tokens over ranks / max time.
 
 --impl reference times the CPU implementation on the host cores (rank 0 only).
---layered times the mixer-layer models instead (llamatov_b200/measure_layered.py), beside the Q8_0 block at equal size.
+--layered times the models made of mixer layers instead (llamatov_b200/measure_layered.py: Pakalix, Nugusun), beside the Q8_0
+block at equal size.
 """
 import argparse
 import ctypes
@@ -332,8 +333,8 @@ def main():
     ap.add_argument("--tp-steps", type=int, default=32)
     ap.add_argument("--config0", action="store_true", help="the single-GEMV case (BASELINE config 0) instead of decode")
     ap.add_argument("--layered", nargs="?", const="0.5b,3b,8b", default=None, metavar="SIZES",
-                    help="prefill / decode throughput and kernel times of the mixer-layer models beside the Q8_0 llama "
-                         "block at equal size, instead of the headline workload")
+                    help="prefill / decode throughput and kernel times of the mixer-layer models (Pakalix, Nugusun) beside the "
+                         "Q8_0 llama block at equal size, instead of the headline workload")
     ap.add_argument("--step-mode", default=None, choices=["pdl", "persistent", "per-op"],
                     help="how the captured decode step is built (default: the engine's default)")
     args = ap.parse_args()

@@ -3,7 +3,8 @@ time of every kernel against its roofline.  `bench.py --layered`; every number i
 after warm-up, weights are random.
 
 A size names width, feed-forward, heads and head size; the mixer model's layers are, in turn, lightning, gla, latent
-attention (window as given) and gla, the llama model has the same number of attention blocks of the same sizes.
+attention (window as given) and gla, the llama model has the same number of attention blocks of the same sizes.  The Pakalix
+model has three Mamba-2 layers (inner size twice the width, heads of 64, state 128) to one of grouped-query attention.
 """
 import ctypes
 
@@ -22,6 +23,12 @@ SIZES = {
     "8b": dict(E=4096, F=14336, H=32, nkv=8, hd=128, rank_a=32, kv_rank=512, rot=64, window=4096, layers=4, V=32768),
 }
 KINDS = ("lightning", "gla", "latent_attention", "gla")
+PAKALIX_KINDS = ("mamba2", "attention", "mamba2", "mamba2")
+
+
+def ssd_sizes(s):
+    """heads, value size, state, groups, taps of the Mamba-2 layers of a size"""
+    return 2 * s["E"] // 64, 64, 128, 1, 4
 
 
 def mixer_model(s, dtype="bfloat16", seed=0):
@@ -61,6 +68,40 @@ def mixer_model(s, dtype="bfloat16", seed=0):
         layers.append({"type": kind, "mixer": m, "mlp": {"kind": "dense", "ff": F}})
     js = {"architecture": "Nugusun", "embedding": {"scale": 1.0}, "layers": layers, "norm": {"eps": 1e-6}, "vocab": V, "width": E}
     cfg = layered.ARCH.config_from_json(js, dtype)
+    return cfg, layered.DenseWeights(w)
+
+
+def pakalix_model(s, dtype="bfloat16", seed=0):
+    """(cfg, w) of the Pakalix model of a size, random weights."""
+    g = torch.Generator(device="cuda").manual_seed(seed)
+    E, F, H, hd, V, G = s["E"], s["F"], s["H"], s["hd"], s["V"], s["nkv"]
+    SH, P, N, SG, taps = ssd_sizes(s)
+
+    def lin(o, i):
+        return (torch.randn(o, i, generator=g, device="cuda") / i ** 0.5).bfloat16().cpu()
+
+    def vec(n, m=0.0):
+        return (m + 0.1 * torch.randn(n, generator=g, device="cuda")).bfloat16().cpu()
+    w = {"embed": lin(V, E), "embed.norm": vec(E), "final.norm": vec(E), "head": lin(V, E)}
+    layers = []
+    for i in range(s["layers"]):
+        kind, p = PAKALIX_KINDS[i % len(PAKALIX_KINDS)], f"l{i}.mix."
+        w[f"l{i}.norm1"] = vec(E)
+        if kind == "attention":
+            m = {"heads": H, "kv_heads": G, "dim": hd, "vdim": hd, "rot": {"base": 10000.0, "dims": hd}, "scale": hd ** -0.5, "softcap": 30.0,
+                 "v_mix": True}
+            w[p + "q"], w[p + "k"], w[p + "v"], w[p + "g"], w[p + "o"] = lin(H * hd, E), lin(G * hd, E), lin(G * hd, E), lin(H, E), lin(E, H * hd)
+            w[p + "q.norm"], w[p + "k.norm"], w[p + "vmix"] = vec(H * hd, 1.0), vec(G * hd, 1.0), torch.tensor(0.4).bfloat16()
+        else:
+            m = {"heads": SH, "groups": SG, "vdim": P, "state": N, "conv": taps, "norm_groups": 1}
+            inner, ch = SH * P, SH * P + 2 * SG * N
+            w[p + "in"], w[p + "conv"], w[p + "conv.b"], w[p + "norm"], w[p + "o"] = lin(inner + ch + SH, E), lin(ch, taps), vec(ch), vec(inner, 1.0), lin(E, inner)
+            w[p + "dt_bias"], w[p + "A_log"], w[p + "D"] = vec(SH, -2.0), vec(SH, 0.5), vec(SH, 1.0)
+        for n, o, k in (("gate", F, E), ("up", F, E), ("down", E, F)):
+            w[f"l{i}.mlp.{n}"] = lin(o, k)
+        layers.append({"type": kind, "mixer": m, "mlp": {"kind": "dense", "ff": F, "limit": 7.0}})
+    js = {"architecture": "Pakalix", "layers": layers, "norm": {"eps": 1e-6}, "residual_mult": 0.25, "vocab": V, "width": E}
+    cfg = layered.PAKALIX.config_from_json(js, dtype)
     return cfg, layered.DenseWeights(w)
 
 
@@ -297,6 +338,8 @@ def kernel_times(s, T, only=None):
         us = _chain_us([lambda: _lib.call("lt_attn_decode_masked", qkv.data_ptr(), kc.data_ptr(), vc.data_ptr(), ln.data_ptr(), yq.data_ptr(), hd, H,
                                           s["nkv"], float(hd ** -0.5), T + 8, st())] * 8)
         add(f"q8 attention token, {T} positions", us, T * 2 * kvw * 4, 0)
+    if want("pakalix"):
+        pakalix_kernels(s, T, add, st)
     # ---- row operators
     if want("norm"):
         n = _copies(T * E * 4)
@@ -311,6 +354,121 @@ def kernel_times(s, T, only=None):
     return out
 
 
+def pakalix_kernels(s, T, add, st):
+    """The kernels of the Pakalix layers; `like` names the kernel of the other mixer model to compare with."""
+    E, F, H, hd, G = s["E"], s["F"], s["H"], s["hd"], s["nkv"]
+    SH, P, N, SG, taps = ssd_sizes(s)
+    dev = dict(device="cuda")
+    bf = lambda *sh: torch.randn(*sh, device="cuda").bfloat16()
+    inner, ch = SH * P, SH * P + 2 * SG * N
+    f32e = torch.zeros(T, max(SH, H), **dev)
+    # ---- linears: (name, rows, K, kind); gate and up rows follow those of the input projection
+    ins = (("in, state space", inner + ch, SH, inner), ("in, attention", (H + 2 * G) * hd, H, H * hd))
+    for name, M, tail, nin in ins:
+        W = [bf(M + tail + 2 * F, E) for _ in range(_copies((M + tail + 2 * F) * E * 2))]
+        X = [bf(T, E) for _ in range(3)]
+        Y, Z = torch.zeros(T, M, dtype=torch.bfloat16, **dev), torch.zeros(T, nin + F, dtype=torch.bfloat16, **dev)
+        e = dense_ops.with_tail(dense_ops.epilogue(segs=[(M, None, 1.0), (M + tail, "sigmoid", 1.0)], tail_from=M), f32e.data_ptr(), tail)
+        n = max(len(W), 3)
+        us = _chain_us([lambda i=i: _lib.call("lt_dn_linear", W[i % len(W)].data_ptr(), E, X[i % 3].data_ptr(), E, Y.data_ptr(), M, 0, M + tail, E, T,
+                                              ctypes.byref(e), 0, st()) for i in range(n)])
+        add(f"linear {name} {M + tail}x{E}, {T} rows", us, (M + tail) * E * 2 + T * E * 2 + T * M * 2, 2.0 * (M + tail) * E * T, "linear qkvg")
+        if name == "in, state space":
+            g = dense_ops.epilogue(_lib.DN_GLU, glu=(_lib.DN_GLU_CLAMPED, 1.702, 7.0))
+            us = _chain_us([lambda i=i: _lib.call("lt_dn_linear", W[i % len(W)].data_ptr() + (M + tail) * E * 2, E, X[i % 3].data_ptr(), E,
+                                                  Z.data_ptr() + nin * 2, nin + F, 0, F, E, T, ctypes.byref(g), 0, st()) for i in range(n)])
+            add(f"linear gate|up clamped {2 * F}x{E}, {T} rows", us, 2 * F * E * 2 + T * E * 2 + T * F * 2, 4.0 * F * E * T, "linear gate|up")
+        x, y, z = torch.randn(E, **dev), torch.zeros(M, dtype=torch.bfloat16, **dev), torch.zeros(F, dtype=torch.bfloat16, **dev)
+        pro = dense_ops.Norm(torch.ones(E), E, E, 1e-6).prologue(x.data_ptr())
+        c = _lib.DnEpilogue.from_buffer_copy(e)
+        c.kind, c.glu_from, c.y2, c.glu_act, c.glu_alpha, c.glu_limit = _lib.DN_STORE_GLU, M + tail, z.data_ptr(), 1, 1.702, 7.0
+        us = _chain_us([lambda i=i: _lib.call("lt_dn_gemv", W[i].data_ptr(), E, y.data_ptr(), 0, M + tail + F, E, ctypes.byref(pro), ctypes.byref(c), st())
+                        for i in range(len(W))])
+        add(f"gemv {name} and gate|up {M + tail + 2 * F}x{E}", us, (M + tail + 2 * F) * E * 2, 0, "gemv gate|up")
+        del W
+        K = nin + F
+        W = [bf(E, K) for _ in range(_copies(E * K * 2))]
+        X = [bf(T, K) for _ in range(3)]
+        R, ls = torch.zeros(T, E, **dev), torch.full((E,), 0.25, **dev)
+        e = dense_ops.epilogue(_lib.DN_RESID, ls=ls)
+        n = max(len(W), 3)
+        us = _chain_us([lambda i=i: _lib.call("lt_dn_linear", W[i % len(W)].data_ptr(), K, X[i % 3].data_ptr(), K, R.data_ptr(), E, 0, E, K, T,
+                                              ctypes.byref(e), 0, st()) for i in range(n)])
+        add(f"linear o and down, {name[4:]} {E}x{K}, {T} rows", us, E * K * 2 + T * K * 2 + T * E * 8, 2.0 * E * K * T, "linear down")
+        o, f = torch.randn(nin, **dev), bf(K)
+        if name == "in, state space":
+            pro = dense_ops.Norm(torch.ones(nin), nin, nin, 1e-6, gate_first=True).prologue(o.data_ptr(), f.data_ptr())
+            pro.n1, pro.x2 = nin, f.data_ptr()
+        else:
+            pro = dense_ops.typed_input(f.data_ptr())
+        us = _chain_us([lambda i=i: _lib.call("lt_dn_gemv", W[i].data_ptr(), K, R.data_ptr(), 0, E, K, ctypes.byref(pro), ctypes.byref(e), st())
+                        for i in range(len(W))])
+        add(f"gemv o and down, {name[4:]} {E}x{K}", us, E * K * 2, 0, "gemv down")
+        del W, X
+    # ---- state space
+    ld = inner + ch
+    ys = [(torch.randn(T, ld, device="cuda") * 0.5).bfloat16() for _ in range(_copies(T * ld * 2))]
+    conv, cb, one, A = torch.randn(taps, ch, **dev), torch.zeros(ch, **dev), torch.ones(SH, **dev), -torch.ones(SH, **dev)
+    desc = _lib.DnSsd(SH, SG, N, P, taps, conv.data_ptr(), cb.data_ptr(), one.data_ptr(), A.data_ptr(), one.data_ptr())
+    ring, u = torch.zeros(taps, ch, dtype=torch.bfloat16, **dev), torch.zeros(T, ch, dtype=torch.bfloat16, **dev)
+    dt, hla, hdt = torch.randn(T, SH, **dev), torch.zeros(T, SH, **dev), torch.zeros(T, SH, **dev)
+    us = _chain_us([lambda y=y_: _lib.call("lt_dn_ssd_rows", y.data_ptr() + inner * 2, ld, dt.data_ptr(), SH, ring.data_ptr(), u.data_ptr(), ch,
+                                           hla.data_ptr(), hdt.data_ptr(), 0, T, 0, ctypes.byref(desc), st()) for y_ in ys])
+    add(f"state-space convolution (2 launches), {ch} channels, {T} rows", us, T * ch * 4 + T * SH * 12, 0, "latent rows")
+    us_ = [(torch.randn(T, ch, device="cuda") * 0.5).bfloat16() for _ in range(_copies(T * ch * 2))]
+    S, o = torch.zeros(SH, P, N, **dev), torch.empty(T, inner, **dev)
+    hdt.fill_(0.05); hla.fill_(-0.05)
+    ws = torch.empty(_lib.dense().lt_dn_recurrence_chunked_ws(T, SH, N, P), **dev)
+    dec = _lib.DnDecay()
+    dec.hla, dec.hdt, dec.D, dec.ldh, dec.per = hla.data_ptr(), hdt.data_ptr(), one.data_ptr(), SH, SH // SG
+    us = _chain_us([lambda x=x_: _lib.call("lt_dn_recurrence_chunked", x.data_ptr() + (inner + SG * N) * 2, x.data_ptr() + inner * 2, x.data_ptr(), ch,
+                                           S.data_ptr(), o.data_ptr(), inner, T, SH, N, P, ctypes.byref(dec), ws.data_ptr(), st()) for x_ in us_])
+    add(f"recurrence state space, {SH} heads of {N}x{P}, {T} rows", us, T * (ch * 2 + inner * 4), 2.0 * T * SH * (2 * N * P + 64 * P) + 2.0 * T * SG * 64 * N,
+        "recurrence lightning")
+    Ss = [torch.zeros(SH, P, N, **dev) for _ in range(_copies(SH * P * N * 4))]
+    ln, tk = torch.full((1,), 100, dtype=torch.int32, **dev), torch.zeros(1, dtype=torch.int32, **dev)
+    us = _chain_us([lambda S=S_: _lib.call("lt_dn_ssd_step", ys[0].data_ptr() + inner * 2, dt.data_ptr(), ring.data_ptr(), S.data_ptr(), o.data_ptr(), 0,
+                                           ln.data_ptr(), tk.data_ptr(), ctypes.byref(desc), st()) for S_ in Ss])
+    add("state-space step, one token", us, 2 * SH * N * P * 4 + ch * taps * 6, 0, "recurrence lightning, one token")
+    os_ = [torch.randn(T, inner, **dev) for _ in range(_copies(T * inner * 4))]
+    nm, X = dense_ops.Norm(torch.ones(inner), inner, inner, 1e-6, gate_first=True), torch.zeros(T, inner + F, dtype=torch.bfloat16, **dev)
+    us = _chain_us([lambda i=i: nm.rows(os_[i].data_ptr(), inner, X.data_ptr(), inner + F, 0, T, inner, gate=ys[i % len(ys)].data_ptr(), ldg=ld)
+                    for i in range(len(os_))])
+    add(f"gated norm rows {T}x{inner}", us, T * inner * 8, 0, "norm rows")
+    del ys, us_, Ss, os_
+    # ---- attention
+    cap, w = T + 64, (H + 2 * G) * hd
+    half = hd // 2
+    freq, qn, kn = torch.rand(half, 2, **dev), torch.ones(H * hd, **dev), torch.ones(G * hd, **dev)
+    freq[:, 1] = 0
+    a = _lib.DnGqa(H, G, hd, hd, hd, H * hd, G * hd, cap, hd ** -0.5, 30.0, 1e-6, 0.4, freq.data_ptr(), qn.data_ptr(), kn.data_ptr())
+    ys = [bf(T, w) for _ in range(_copies(T * w * 2))]
+    kc, vc, vf = bf(cap, G * hd), bf(cap, G * hd), bf(T, G * hd)
+    gate, out = torch.rand(T, H, **dev), torch.zeros(T, H * hd, dtype=torch.bfloat16, **dev)
+    us = _chain_us([lambda y=y_: _lib.call("lt_dn_gqa_rows", y.data_ptr(), w, kc.data_ptr(), vc.data_ptr(), vf.data_ptr(), 0, 0, T, 0, ctypes.byref(a), st())
+                    for y_ in ys])
+    add(f"grouped attention rows, {T} rows", us, T * (2 * H + 5 * G) * hd * 2, 0, "latent rows")
+    for cap_on in (True, False):
+        a.softcap = 30.0 if cap_on else 0.0
+        us = _chain_us([lambda y=y_: _lib.call("lt_dn_gqa_attn", y.data_ptr(), w, kc.data_ptr(), vc.data_ptr(), gate.data_ptr(), H, out.data_ptr(), H * hd, 0,
+                                               T, 0, ctypes.byref(a), st()) for y_ in ys[:4]])
+        add(f"grouped attention, {H} heads on {G}, {T} rows" + ("" if cap_on else ", no cap"), us, T * (2 * H + 2 * G) * hd * 2,
+            2.0 * (T * (T + 1) // 2) * H * 2 * hd, "latent window attention")
+    a.softcap = 30.0
+    kcs, vcs = [bf(cap, G * hd) for _ in range(24)], [bf(cap, G * hd) for _ in range(24)]
+    tk = torch.zeros(_lib.dense().lt_dn_gqa_step_tickets(H, G), dtype=torch.int32, **dev)
+    splits = max(1, 296 // (tk.numel() - 1))
+    splits = min(splits, (cap + 15) // 16)
+    ws = torch.empty(_lib.dense().lt_dn_gqa_step_ws(H, hd, splits), **dev)
+    lens = [torch.full((1,), T, dtype=torch.int32, **dev) for _ in range(24)]
+
+    def one_step(i):
+        _lib.call("lt_dn_gqa_step", ys[0].data_ptr(), kcs[i % 24].data_ptr(), vcs[i % 24].data_ptr(), vf.data_ptr(), 0, gate.data_ptr(), out.data_ptr(), 0,
+                  lens[i % 24].data_ptr(), ctypes.byref(a), splits, ws.data_ptr(), tk.data_ptr(), st())
+    us = _chain_us([lambda i=i: one_step(i) for i in range(24)])
+    add(f"grouped attention step, {T} positions", us, T * 2 * G * hd * 2, 0, "latent step")
+
+
 def run(sizes=("0.5b", "3b", "8b"), tokens=2048, steps=64, kernels=True, models=True, only=None):
     res = []
     hbm, tf, src = peaks()
@@ -318,7 +476,7 @@ def run(sizes=("0.5b", "3b", "8b"), tokens=2048, steps=64, kernels=True, models=
         s = SIZES[name]
         r = {"size": name, **{k: s[k] for k in ("E", "F", "H", "hd", "layers", "window", "kv_rank")}, "prompt": tokens}
         if models:
-            for label, make in (("mixers_bf16", mixer_model), ("llama_q8", llama_model)):
+            for label, make in (("pakalix_bf16", pakalix_model), ("mixers_bf16", mixer_model), ("llama_q8", llama_model)):
                 dr.reset_engine_state(); dr.apply_production_profile()
                 cfg, w = make(s)
                 fused = dr._FUSED_STEP
@@ -328,7 +486,7 @@ def run(sizes=("0.5b", "3b", "8b"), tokens=2048, steps=64, kernels=True, models=
                     r[label] = run_model(cfg, w, tokens, steps)
                 finally:
                     dr._FUSED_STEP = fused
-                if label == "mixers_bf16":
+                if label != "llama_q8":
                     wb = sum(L.numel() * 2 for k, L in w.items() if k != "embed")
                 else:
                     wb = sum(q.N * q.K * 34 // 32 for q in w.values() if isinstance(q, Q8Weight))
