@@ -3,19 +3,16 @@
 //     dS        = sum_j (k_j e^(b_end - b_j)) v_j^T                            k_chunk_state, every chunk at once
 //     S_next    = e^(b_end) S + dS                                            k_chunk_scan, element by element
 //     o_t       = (q_t e^(b_t))^T S + sum_(j <= t) (q_t . k_j e^(b_t - b_j)) v_j   k_chunk_out, every chunk at once
-// (state-space form, MODE_HEAD: a decay per token and head, k_j carries the step size dt_j, o_t gains D v_t, and neighbouring
-// heads share q and k).  q, k and v are bf16 as they are; whatever a decay has touched, the state and the weights of the last sum enter their
+// q, k and v are bf16 as they are; whatever a decay has touched, the state and the weights of the last sum enter their
 // products as a sum of two bf16 (16 significant bits).  No exponential grows: the weights are formed in blocks of 16
 // tokens, decays measured from the start of the query's block, (q_t e^(b_t - r)) . (k_j e^(r - b_j)); inside the block
 // the second exponent is positive, and where it could leave a safe range the block's weights are summed pair by pair.
+#include "lt_dn_chunk.cuh"
 #include "lt_dn_mma.cuh"
 
 namespace lt {
 namespace dn {
 
-constexpr int CH = 64;
-enum { MODE_CONST = 0, MODE_LOG = 1, MODE_HEAD = 2 };
-constexpr float LOG2E = 1.4426950408889634f;   // the kernels keep log decays to base 2
 constexpr float SAFE_EXP = 86.0f;              // of 2 (e^60)
 
 struct ChunkP {
@@ -25,8 +22,6 @@ struct ChunkP {
     const float* decay;
     const float* la;
     int ldla;
-    const float *hla, *hdt, *D;
-    int ldh, per;                 // per: consecutive heads that share q and k
 };
 
 // rows [t0, t0 + 64) x n columns of a bf16 matrix into shared memory, zero rows past T
@@ -52,7 +47,7 @@ __device__ __forceinline__ void load_logs(float* dst, int stride, const float* l
 
 // ---------------------------------------------------------------------------- dS of every chunk
 
-template <int MODE>
+template <bool LOG>
 __global__ void __launch_bounds__(256) k_chunk_state(const __grid_constant__ ChunkP P) {
     extern __shared__ __align__(16) unsigned char smem[];
     const int ks = P.dp + 8, vs = P.dvp + 8;      // an odd number of 16-byte units
@@ -61,10 +56,9 @@ __global__ void __launch_bounds__(256) k_chunk_state(const __grid_constant__ Chu
     bf16* sv = sl + CH * ks;
     float* sla = (float*)(sv + CH * vs);
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-    constexpr bool LOG = MODE == MODE_LOG;
     const int chunk = blockIdx.x, h = blockIdx.y, t0 = chunk * CH, n = min(CH, P.T - t0);
 
-    load_tile(sh, ks, P.k + (long)(MODE == MODE_HEAD ? h / P.per : h) * P.dp, P.ld, t0, P.T, P.dp);
+    load_tile(sh, ks, P.k + (long)h * P.dp, P.ld, t0, P.T, P.dp);
     load_tile(sv, vs, P.v + (long)h * P.dvp, P.ld, t0, P.T, P.dvp);
     if (LOG) load_logs(sla, P.dp, P.la + (long)h * P.dp, P.ldla, t0, P.T, P.dp);
     __syncthreads();
@@ -84,20 +78,9 @@ __global__ void __launch_bounds__(256) k_chunk_state(const __grid_constant__ Chu
             if (seg == 0) P.dend[((long)chunk * P.H + h) * P.dp + c] = exp2f(s);
         }
     } else {
+        const float lam = P.decay[h];
         float* pw = sla;
-        if (MODE == MODE_HEAD) {
-            float* sl2 = sla + CH;
-            if (tid < CH) sl2[tid] = tid < n ? P.hla[(long)(t0 + tid) * P.ldh + h] * LOG2E : 0.0f;
-            __syncthreads();
-            if (tid < CH) {
-                float s = 0.0f;
-                for (int j = CH - 1; j > tid; j--) s += sl2[j];
-                pw[tid] = tid < n ? exp2f(s) * P.hdt[(long)(t0 + tid) * P.ldh + h] : 0.0f;
-                if (tid == 0) P.dend[(long)chunk * P.H + h] = exp2f(s + sl2[0]);
-            }
-        } else if (tid < CH) {
-            pw[tid] = tid < n ? powf(P.decay[h], (float)(n - 1 - tid)) : 0.0f;
-        }
+        if (tid < CH) pw[tid] = tid < n ? powf(lam, (float)(n - 1 - tid)) : 0.0f;
         __syncthreads();
         for (int e = tid; e < CH * P.dp; e += 256) {
             const int j = e / P.dp, c = e - j * P.dp;
@@ -148,7 +131,7 @@ __global__ void __launch_bounds__(256) k_chunk_state(const __grid_constant__ Chu
 // ---------------------------------------------------------------------------- states between chunks
 
 // Replaces dS of each chunk by the state the chunk starts from, four channels at a time as {4 x bf16 hi, 4 x bf16 lo}.
-template <int MODE>
+template <bool LOG>
 __global__ void __launch_bounds__(256) k_chunk_scan(const __grid_constant__ ChunkP P) {
     const int nq = P.dp >> 2;
     const long i = (long)blockIdx.x * 256 + threadIdx.x, per = (long)P.H * P.dvp * nq;
@@ -158,7 +141,7 @@ __global__ void __launch_bounds__(256) k_chunk_scan(const __grid_constant__ Chun
     float4* w = (float4*)P.ws + i;
     float4 s = *S;
     float full = 0.0f, tail = 0.0f;
-    if (MODE == MODE_CONST) {
+    if (!LOG) {
         full = powf(P.decay[h], (float)CH);
         tail = powf(P.decay[h], (float)(P.T - (P.nchunk - 1) * CH));
     }
@@ -171,9 +154,9 @@ __global__ void __launch_bounds__(256) k_chunk_scan(const __grid_constant__ Chun
         split2(s.z, s.w, h1, l1);
         *(uint4*)(w + (long)c * per) = make_uint4(h0, h1, l0, l1);
         float4 a;
-        if (MODE == MODE_LOG) a = *(const float4*)(P.dend + ((long)c * P.H + h) * P.dp + cq * 4);
+        if (LOG) a = *(const float4*)(P.dend + ((long)c * P.H + h) * P.dp + cq * 4);
         else {
-            const float f = MODE == MODE_HEAD ? P.dend[(long)c * P.H + h] : c + 1 < P.nchunk ? full : tail;
+            const float f = c + 1 < P.nchunk ? full : tail;
             a = make_float4(f, f, f, f);
         }
         s.x = fmaf(a.x, s.x, d.x); s.y = fmaf(a.y, s.y, d.y);
@@ -196,9 +179,8 @@ __device__ __forceinline__ Quad load_quad(const bf16* p) {
     return q;
 }
 
-template <int MODE>
+template <bool LOG>
 __global__ void __launch_bounds__(256, 2) k_chunk_out(const __grid_constant__ ChunkP P) {
-    constexpr bool LOG = MODE == MODE_LOG;
     extern __shared__ __align__(16) unsigned char smem[];
     const int qs = ((P.dp + 63) & ~63) + 16;       // bf16 row stride: rows 8 banks apart for 8-byte reads
     const int bs = ((P.dp + 31) & ~31) + 16;       // fp32 row stride: rows 16 banks apart for 16-byte reads
@@ -211,19 +193,15 @@ __global__ void __launch_bounds__(256, 2) k_chunk_out(const __grid_constant__ Ch
     bf16* sAl = sAh + CH * as;
     // LOG: sums of the log decays per channel, inside each block of 16 tokens (so that a difference inside a block does
     // not inherit the rounding of what came before), then sp[0..3]: what the blocks before block I add up to.
-    // MODE_CONST: powers of the head's decay.  MODE_HEAD: running sums of the log decays (double, so that differences are
-    // exact), then the step sizes.
+    // Else: powers of the head's decay.
     float* sb = (float*)(sAl + CH * as);
     float* sp = sb + CH * bs;
-    double* sd = (double*)sb;
-    float* sdt = (float*)(sd + CH);
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tg = lane & 3;
     const int chunk = blockIdx.x, h = blockIdx.y, t0 = chunk * CH;
     const int dk = (P.dp + 15) & ~15;              // contraction length; rows are zero past dp
 
-    const int hq = MODE == MODE_HEAD ? h / P.per : h;
-    load_tile(sq, qs, P.q + (long)hq * P.dp, P.ld, t0, P.T, P.dp);
-    load_tile(sk, qs, P.k + (long)hq * P.dp, P.ld, t0, P.T, P.dp);
+    load_tile(sq, qs, P.q + (long)h * P.dp, P.ld, t0, P.T, P.dp);
+    load_tile(sk, qs, P.k + (long)h * P.dp, P.ld, t0, P.T, P.dp);
     load_tile(sv, vs, P.v + (long)h * P.dvp, P.ld, t0, P.T, P.dvp);
     for (int e = tid; e < CH; e += 256) {
         *(uint4*)(sq + e * qs + P.dp) = make_uint4(0, 0, 0, 0);
@@ -249,19 +227,6 @@ __global__ void __launch_bounds__(256, 2) k_chunk_out(const __grid_constant__ Ch
                 sp[I * bs + c] = s;
                 s += sb[(I * 16 + 15) * bs + c];
             }
-        }
-    } else if (MODE == MODE_HEAD) {
-        float* sl = sdt + CH;
-        if (tid < CH) {
-            const bool ok = t0 + tid < P.T;
-            sl[tid] = ok ? P.hla[(long)(t0 + tid) * P.ldh + h] * LOG2E : 0.0f;
-            sdt[tid] = ok ? P.hdt[(long)(t0 + tid) * P.ldh + h] : 0.0f;
-        }
-        __syncthreads();
-        if (tid < CH) {
-            double s = 0.0;
-            for (int j = 0; j <= tid; j++) s += (double)sl[j];
-            sd[tid] = s;
         }
     } else if (tid <= CH) {
         sb[tid] = powf(P.decay[h], (float)tid);
@@ -337,13 +302,9 @@ __global__ void __launch_bounds__(256, 2) k_chunk_out(const __grid_constant__ Ch
         for (int i = 0; i < 4; i += 2) {
             const int t = tq + 8 * (i >> 1), j = J * 16 + half * 8 + 2 * tg;
             float x = j <= t ? acc[i] : 0.0f, y = j + 1 <= t ? acc[i + 1] : 0.0f;
-            if (MODE == MODE_CONST) {
+            if (!LOG) {
                 x *= sb[max(t - j, 0)];
                 y *= sb[max(t - j - 1, 0)];
-            }
-            if (MODE == MODE_HEAD) {
-                x *= exp2f(fminf((float)(sd[t] - sd[j]), 0.0f)) * sdt[j];
-                y *= exp2f(fminf((float)(sd[t] - sd[j + 1]), 0.0f)) * sdt[j + 1];
             }
             unsigned hi, lo;
             split2(x, y, hi, lo);
@@ -402,8 +363,7 @@ __global__ void __launch_bounds__(256, 2) k_chunk_out(const __grid_constant__ Ch
 #pragma unroll
             for (int m = 0; m < 2; m++) {
                 const int t = (mt + m) * 16 + g;
-                const float fa = MODE == MODE_HEAD ? exp2f((float)sd[t]) : sb[t + 1];
-                const float fb = MODE == MODE_HEAD ? exp2f((float)sd[t + 8]) : sb[t + 9];
+                const float fa = sb[t + 1], fb = sb[t + 9];
 #pragma unroll
                 for (int n = 0; n < 4; n++) {
                     acc[m][n][0] *= fa; acc[m][n][1] *= fa;
@@ -437,43 +397,34 @@ __global__ void __launch_bounds__(256, 2) k_chunk_out(const __grid_constant__ Ch
                 const int t = t0 + (mt + m) * 16 + g + r * 8;
                 if (t >= P.T) continue;
                 float* o = P.o + (long)t * P.ldo + (long)h * P.dvp;
-                const float D = MODE == MODE_HEAD ? P.D[h] : 0.0f;
-                const bf16* vr = sv + (t - t0) * vs;
 #pragma unroll
                 for (int n = 0; n < 4; n++) {
                     const int v = v0 + n * 8 + tg * 2;
-                    if (v >= P.dvp) continue;
-                    float2 y = make_float2(acc[m][n][2 * r], acc[m][n][2 * r + 1]);
-                    if (MODE == MODE_HEAD) {
-                        y.x = fmaf(D, to_f(vr[v]), y.x);
-                        y.y = fmaf(D, to_f(vr[v + 1]), y.y);
-                    }
-                    *(float2*)(o + v) = y;
+                    if (v < P.dvp) *(float2*)(o + v) = make_float2(acc[m][n][2 * r], acc[m][n][2 * r + 1]);
                 }
             }
     }
 }
 
-template <int MODE>
+template <bool LOG>
 static int launch_chunked(const ChunkP& P, cudaStream_t s) {
-    constexpr bool LOG = MODE == MODE_LOG;
-    const size_t sm1 = (size_t)CH * (2 * (P.dp + 8) + P.dvp + 8) * 2 + (LOG ? (size_t)CH * P.dp * 4 : 2 * CH * 4);
+    const size_t sm1 = (size_t)CH * (2 * (P.dp + 8) + P.dvp + 8) * 2 + (LOG ? (size_t)CH * P.dp * 4 : CH * 4);
     const int qs = ((P.dp + 63) & ~63) + 16, bs = ((P.dp + 31) & ~31) + 16;
-    const size_t sm2 = (size_t)CH * (2 * qs + P.dvp + 8 + 2 * (CH + 8)) * 2 + (LOG ? (size_t)(CH + 4) * bs * 4 : CH * 16);
+    const size_t sm2 = (size_t)CH * (2 * qs + P.dvp + 8 + 2 * (CH + 8)) * 2 + (LOG ? (size_t)(CH + 4) * bs * 4 : (CH + 4) * 4);
     LT_REQUIRE(sm1 <= 220 * 1024 && sm2 <= 220 * 1024, "lt_dn_recurrence_chunked: head sizes %d, %d need too much shared memory", P.dp, P.dvp);
     static PerDeviceOnce once;
     if (once.first()) {
-        LT_CUDA(cudaFuncSetAttribute(k_chunk_state<MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
-        LT_CUDA(cudaFuncSetAttribute(k_chunk_out<MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+        LT_CUDA(cudaFuncSetAttribute(k_chunk_state<LOG>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
+        LT_CUDA(cudaFuncSetAttribute(k_chunk_out<LOG>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
     }
-    k_chunk_state<MODE><<<dim3(P.nchunk, P.H), 256, sm1, s>>>(P);
+    k_chunk_state<LOG><<<dim3(P.nchunk, P.H), 256, sm1, s>>>(P);
     int rc = check_launch("lt_dn_recurrence_chunked (state)");
     if (rc != LT_OK) return rc;
     const long per = (long)P.H * P.dvp * (P.dp >> 2);
-    k_chunk_scan<MODE><<<(unsigned)((per + 255) / 256), 256, 0, s>>>(P);
+    k_chunk_scan<LOG><<<(unsigned)((per + 255) / 256), 256, 0, s>>>(P);
     rc = check_launch("lt_dn_recurrence_chunked (scan)");
     if (rc != LT_OK) return rc;
-    k_chunk_out<MODE><<<dim3(P.nchunk, P.H), 256, sm2, s>>>(P);
+    k_chunk_out<LOG><<<dim3(P.nchunk, P.H), 256, sm2, s>>>(P);
     return check_launch("lt_dn_recurrence_chunked (out)");
 }
 
@@ -485,7 +436,7 @@ using namespace lt::dn;
 
 extern "C" long lt_dn_recurrence_chunked_ws(int T, int H, int dp, int dvp) {
     const long n = (T + CH - 1) / CH;
-    return n * H * dp * ((long)dvp + 1);
+    return n * H * ((dp + 15) & ~15) * ((long)dvp + 1);
 }
 
 extern "C" int lt_dn_recurrence_chunked(const void* q, const void* k, const void* v, int ld, float* S, float* o, int ldo, int T, int H,
@@ -498,15 +449,20 @@ extern "C" int lt_dn_recurrence_chunked(const void* q, const void* k, const void
     LT_REQUIRE(ld % 8 == 0 && ldo % 2 == 0 && aligned16(q) && aligned16(k) && aligned16(v) && aligned16(S) && aligned16(o) && aligned16(ws),
                "lt_dn_recurrence_chunked: alignment");
     LT_REQUIRE(h_decay->decay || !h_decay->la || (h_decay->ldla % 4 == 0 && aligned16(h_decay->la)), "lt_dn_recurrence_chunked: alignment of the logarithms");
+    if (!h_decay->decay && !h_decay->la) {
+        SsdChunkP Q = {};
+        Q.q = (const bf16*)q; Q.k = (const bf16*)k; Q.v = (const bf16*)v; Q.S = S; Q.o = o; Q.ws = ws;
+        Q.hla = h_decay->hla; Q.hdt = h_decay->hdt; Q.D = h_decay->D; Q.ldh = h_decay->ldh; Q.per = h_decay->per;
+        LT_REQUIRE(Q.hdt && Q.D && Q.ldh >= H && Q.per > 0 && H % Q.per == 0,
+                   "lt_dn_recurrence_chunked: step sizes, D, or %d heads in groups of %d", H, Q.per);
+        Q.ld = ld; Q.ldo = ldo; Q.T = T; Q.H = H; Q.dp = dp; Q.dvp = dvp; Q.nchunk = (T + CH - 1) / CH;
+        return launch_ssd_chunked(Q, (cudaStream_t)stream);
+    }
     ChunkP P = {};
     P.q = (const bf16*)q; P.k = (const bf16*)k; P.v = (const bf16*)v; P.S = S; P.o = o; P.ld = ld; P.ldo = ldo;
     P.T = T; P.H = H; P.dp = dp; P.dvp = dvp; P.nchunk = (T + CH - 1) / CH;
     P.ws = ws; P.dend = ws + (long)P.nchunk * H * dp * dvp;
     P.decay = h_decay->decay; P.la = h_decay->la; P.ldla = h_decay->ldla;
-    if (P.decay) return launch_chunked<MODE_CONST>(P, (cudaStream_t)stream);
-    if (P.la) return launch_chunked<MODE_LOG>(P, (cudaStream_t)stream);
-    P.hla = h_decay->hla; P.hdt = h_decay->hdt; P.D = h_decay->D; P.ldh = h_decay->ldh; P.per = h_decay->per;
-    LT_REQUIRE(P.hdt && P.D && P.ldh >= H && P.per > 0 && H % P.per == 0,
-               "lt_dn_recurrence_chunked: step sizes, D, or %d heads in groups of %d", H, P.per);
-    return launch_chunked<MODE_HEAD>(P, (cudaStream_t)stream);
+    if (P.decay) return launch_chunked<false>(P, (cudaStream_t)stream);
+    return launch_chunked<true>(P, (cudaStream_t)stream);
 }

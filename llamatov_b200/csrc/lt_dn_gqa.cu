@@ -207,6 +207,16 @@ __global__ void __launch_bounds__(GT) k_gqa_step(const __grid_constant__ GqaStep
 
         // ---- queries of this CTA; the new key and value where the range ends at the new position
         const T* row = (const T*)P.y;
+        for (int e = tid * N; e < nh * A.dp; e += GT * N) {      // query times norm weight, before the norm is known
+            float f[N];
+            Vec<T>::unpack(*(const uint4*)(row + (long)h0 * A.dp + e), f);
+            const float4* w = (const float4*)(A.qnorm + (long)h0 * A.dp + e);
+#pragma unroll
+            for (int i = 0; i < N / 4; i++) {
+                const float4 x = w[i];
+                *(float4*)(sQ + e + 4 * i) = make_float4(f[4 * i] * x.x, f[4 * i + 1] * x.y, f[4 * i + 2] * x.z, f[4 * i + 3] * x.w);
+            }
+        }
         for (int i = tid; i < half; i += GT) rotation(pos, ((const float2*)A.freq)[i], sc[i], ss[i]);
         const float a = warp_sum(square_sum(row, nq, tid, GT)), b = own ? warp_sum(square_sum(row + nq, nk, tid, GT)) : 0.0f;
         if (lane == 0) {
@@ -221,7 +231,19 @@ __global__ void __launch_bounds__(GT) k_gqa_step(const __grid_constant__ GqaStep
             ks += sred[1][i];
         }
         const float qi = 1.0f / sqrtf(qs / (float)A.qcount + A.eps), ki = 1.0f / sqrtf(ks / (float)A.kcount + A.eps);
-        // element j of a normed, rotated head
+        for (int e = tid; e < nh * (A.dp - half); e += GT) {     // half pairs that rotate, then the rest of the head
+            const int h = e / (A.dp - half), i = e - h * (A.dp - half);
+            float* x = sQ + h * A.dp + i;
+            const float u = x[i < half ? 0 : half] * qi;
+            if (i < half) {
+                const float z = x[half] * qi;
+                x[0] = to_f(from_f<T>(u * sc[i] - z * ss[i]));
+                x[half] = to_f(from_f<T>(z * sc[i] + u * ss[i]));
+            } else {
+                x[half] = to_f(from_f<T>(u));
+            }
+        }
+        // element j of the normed, rotated key
         auto turned = [&](const T* x, const float* w, float inv, int j) {
             const float u = to_f(x[j]) * inv * w[j];
             if (j >= A.rot) return u;
@@ -229,11 +251,6 @@ __global__ void __launch_bounds__(GT) k_gqa_step(const __grid_constant__ GqaStep
             const float z = to_f(x[o]) * inv * w[o];
             return j < half ? u * sc[i] - z * ss[i] : u * sc[i] + z * ss[i];
         };
-        for (int e = tid; e < SH * A.dp; e += GT) {
-            const int h = e / A.dp, j = e - h * A.dp;
-            const long o = (long)(h0 + min(h, nh - 1)) * A.dp;
-            sQ[e] = to_f(from_f<T>(turned(row + o, A.qnorm + o, qi, j)));
-        }
         if (own) {
             T* kr = (T*)P.kc + (long)pos * nk + (long)g * A.dp;
             T* vr = (T*)P.vc + (long)pos * nv + (long)g * A.dvp;
@@ -420,7 +437,7 @@ __global__ void __launch_bounds__(GT) k_gqa_step(const __grid_constant__ GqaStep
         const int h = e / nq4, c = (e - h * nq4) * 4;
         const float* u = P.pu + (long)(h0 + h) * A.dvp + c;
         float4 o = make_float4(0, 0, 0, 0);
-#pragma unroll 8
+#pragma unroll 16
         for (int s = 0; s < active; s++) {
             const float4 x = __ldcg((const float4*)(u + (long)s * A.H * A.dvp));
             const float w = sw[h * active + s];
@@ -484,7 +501,7 @@ extern "C" int lt_dn_gqa_step(const void* y, void* kc, void* vc, void* vfirst, i
     LT_REQUIRE(y && kc && vc && out && len && ws && tickets, "lt_dn_gqa_step: null pointer");
     LT_REQUIRE(splits > 0 && splits <= 1024, "lt_dn_gqa_step: splits=%d", splits);
     LT_REQUIRE(h_a->dvp <= 4 * GT, "lt_dn_gqa_step: value size %d of a head is above %d", h_a->dvp, 4 * GT);
-    LT_REQUIRE(aligned16(y) && aligned16(kc) && aligned16(vc) && aligned16(ws), "lt_dn_gqa_step: pointers must be 16-byte aligned");
+    LT_REQUIRE(aligned16(y) && aligned16(kc) && aligned16(vc) && aligned16(ws) && aligned16(h_a->qnorm), "lt_dn_gqa_step: pointers must be 16-byte aligned");
     GqaStepP P = {};
     P.y = y; P.kc = kc; P.vc = vc; P.vfirst = vfirst; P.gate = gate; P.out = out; P.len = len; P.tickets = tickets;
     P.status = device_status_ptr();

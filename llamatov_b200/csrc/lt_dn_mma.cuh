@@ -1,5 +1,5 @@
 // Warp-level tensor-core helpers of the dense kernels (mma.sync m16n8k16, bf16 operands, fp32 accumulation) and the
-// asynchronous 16-byte copy into shared memory.
+// asynchronous copies of 16 and 4 bytes into shared memory.
 #pragma once
 #include "lt_dn_common.cuh"
 
@@ -10,6 +10,10 @@ __device__ __forceinline__ unsigned s_u32(const void* p) { return (unsigned)__cv
 __device__ __forceinline__ void cp16(void* dst, const void* src, bool ok) {
     const int n = ok ? 16 : 0;
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(s_u32(dst)), "l"(src), "r"(n) : "memory");
+}
+__device__ __forceinline__ void cp4(void* dst, const void* src, bool ok) {
+    const int n = ok ? 4 : 0;
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(s_u32(dst)), "l"(src), "r"(n) : "memory");
 }
 __device__ __forceinline__ void ldsm4(unsigned (&r)[4], const void* p) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"

@@ -457,8 +457,7 @@ def pakalix_kernels(s, T, add, st):
     a.softcap = 30.0
     kcs, vcs = [bf(cap, G * hd) for _ in range(24)], [bf(cap, G * hd) for _ in range(24)]
     tk = torch.zeros(_lib.dense().lt_dn_gqa_step_tickets(H, G), dtype=torch.int32, **dev)
-    splits = max(1, 296 // (tk.numel() - 1))
-    splits = min(splits, (cap + 15) // 16)
+    splits = max(1, min(74, 296 // (tk.numel() - 1)))
     ws = torch.empty(_lib.dense().lt_dn_gqa_step_ws(H, hd, splits), **dev)
     lens = [torch.full((1,), T, dtype=torch.int32, **dev) for _ in range(24)]
 

@@ -311,7 +311,7 @@ class GroupedAttentionMixer:
         self.desc = _lib.DnGqa(H, G, self.dp, self.dvp, rot["dims"], H * d, G * d, 0, float(m["scale"]), float(m.get("softcap") or 0.0),
                                cfg["norm_eps"], vmix, *[t.data_ptr() for t in self.keep])
         self.tickets = _lib.dense().lt_dn_gqa_step_tickets(H, G)
-        self.splits = max(1, 2 * self.SMS // (self.tickets - 1))
+        self.splits = max(1, min(74, 2 * self.SMS // (self.tickets - 1)))
         pk.want(ws=_lib.dense().lt_dn_gqa_step_ws(H, self.dvp, self.splits), tickets=self.tickets, vfirst=nv if self.mix else 0)
 
     def new_cache(self, cfg, max_rows):
